@@ -250,6 +250,13 @@ void rotor_b200_model_destroy(void* handle);
 int rotor_b200_model_forward(void* handle, const int64_t* ids, int batch, int seq, int past_len,
                              int logits_mode, float* logits, int64_t* next_ids, void* stream);
 
+/* The same over ids int64 [batch][seq] with logits of selected rows only: `rows` is a HOST array of
+ * nrows row numbers (sequence * seq + position) below batch * seq, logits float32 [nrows][vocab]
+ * (device).  nrows 0 runs the tokens through the caches and computes no logits.  No counterpart in the
+ * reference, which computes every position. */
+int rotor_b200_model_forward_rows(void* handle, const int64_t* ids, int batch, int seq, int past_len,
+                                  const int32_t* rows, int nrows, float* logits, void* stream);
+
 /* Device-resident greedy generation, the cached loop of TextGenerator.generate
  * (src/rotor/generation.py:220-279): begin() seeds the loop with the token picked after the
  * prompt; steps() runs n one-token forwards, each feeding its greedy pick to the next and
@@ -273,6 +280,75 @@ int rotor_b200_model_forward_ragged(void* handle, const int64_t* ids, int batch,
                                     int logits_mode, float* logits, int64_t* next_ids, void* stream);
 int rotor_b200_model_decode_begin_ragged(void* handle, const int64_t* first_ids, int batch, const int32_t* lens,
                                          void* stream);
+
+/* ---------------------------------------------------------------- layer-described decoders
+ * Decoders that no fixed block shape covers: every layer has its own sizes, a layer may run several
+ * times in a row (each run with its own cache), the residual is a set of streams with learned
+ * connections, attention takes a distance bias and a chunk mask.  A handle made here is used through
+ * the rotor_b200_model_* entry points above like a ternary model's (forward, forward_ragged,
+ * forward_rows, decode_*, read_tokens, position, destroy); it is causal, single-GPU, and
+ * forward_hidden does not take it.  No counterpart in the reference.
+ *
+ * Matrices are bf16, row major, row stride = columns rounded up to 64, pad columns zero; vectors
+ * are float32, `width` vectors padded with zeros to that stride as well.  f32 != 0: activations,
+ * caches and every product in float32 on the FP32 pipe; else bf16 with float32 accumulation, while
+ * the residual streams, norms, scores and softmax stay float32. */
+typedef struct rotor_b200_decoder_config {
+    int32_t vocab_size, width, streams, n_layers, n_runs;
+    int32_t f32;
+    float eps;            /* of every norm, the unit norm of queries and keys included */
+    int32_t max_batch, max_seq, max_rows;
+} rotor_b200_decoder_config;
+
+typedef struct rotor_b200_decoder_layer {
+    int32_t heads, kv_heads, dim, vdim;  /* query head h reads KV head h / (heads / kv_heads) */
+    int32_t unit_qk;      /* queries and keys divided by their root mean square over dim */
+    int32_t chunk;        /* > 0: position i sees j <= i with j / chunk == i / chunk; 0: every j <= i */
+    int32_t ff;           /* 0: no feed-forward (its pointers unused) */
+    float scale;          /* score = (q . k) scale - slope (i - j) */
+    const float* slopes;  /* [heads], or NULL for no distance bias */
+    const void* qkv;      /* [heads dim + kv_heads dim + kv_heads vdim][width] */
+    const void* o;        /* [width][heads vdim] */
+    const void* gate_up;  /* [2 ff][width]: gate rows, then up rows; gelu (tanh form) of the gate times up */
+    const void* down;     /* [width][ff] */
+    const float *norm1, *norm2;
+    /* connections of the two sublayers: in [streams], out [streams], mix [from][to] */
+    const float *hc1_in, *hc1_out, *hc1_mix, *hc2_in, *hc2_out, *hc2_mix;
+} rotor_b200_decoder_layer;
+
+/* One run of a layer.  Caches: [max_batch][kv_heads][max_seq][dim rounded up to 8] (vdim for v), bf16 or
+ * float32, zero-filled by the caller before first use. */
+typedef struct rotor_b200_decoder_run {
+    int32_t layer;
+    void* k_cache;
+    void* v_cache;
+} rotor_b200_decoder_run;
+
+/* embed: bf16 [vocab][width rounded up to 64]; head: bf16 [vocab][width rounded up to 256]. */
+size_t rotor_b200_decoder_workspace_bytes(const rotor_b200_decoder_config* cfg, const rotor_b200_decoder_layer* layers);
+int rotor_b200_decoder_create(const rotor_b200_decoder_config* cfg, const rotor_b200_decoder_layer* layers,
+                              const rotor_b200_decoder_run* runs, const void* embed, const void* head,
+                              const float* final_norm, void* workspace, size_t workspace_bytes, void** handle);
+
+/* The decoders' mechanisms one by one, through the kernels the model calls.
+ *  stream_stage: x_out_t = sum_s mix[s][t] x_in_s + out[t] y for every stream t (with ids: x_out_t =
+ *    embed[id]), u = sum_s in[s] x_out_s (in NULL: plain sum), h = u / sqrt(mean(u^2) + eps) * norm.
+ *    x float32 [rows][streams][n rounded up to 64], y and h [rows][n rounded up to 64]; h bf16 or float32.
+ *  dense_linear: y = x w^T (float32) or, gated, gelu(x w_gate^T) (x w_up^T) in the type of x; row strides
+ *    rounded up to 64; scratch float32 [rows][2 n] for gated float32 products.
+ *  bias_attention: raw projections float32 [rows][q | k | v, rounded up to 64] of `seq` tokens per
+ *    sequence behind past_len (device, [batch]) cached ones: appends keys and values, writes the
+ *    attention rows [rows][heads vdim rounded up to 64].  Reads the head sizes and constants of
+ *    `layer`; row_kernel != 0 keeps prompts off the tensor-core kernel; q_scratch bf16
+ *    [rows][heads][dim rounded up to 8]. */
+int rotor_b200_stream_stage(const int64_t* ids, const void* embed, int vocab, const float* x_in, float* x_out, const float* y,
+                            const float* mix, const float* out, const float* in, const float* norm, float eps, int rows,
+                            int streams, int n, void* h, int h_f32, void* stream);
+int rotor_b200_dense_linear(const void* w, int n, int k, const void* x, int rows, int f32, int gated, void* y, float* scratch,
+                            void* stream);
+int rotor_b200_bias_attention(const rotor_b200_decoder_layer* layer, float eps, int f32, const float* qkv, int batch, int seq,
+                              const int32_t* past_len, int max_seq, void* k_cache, void* v_cache, void* out, int row_kernel,
+                              void* q_scratch, void* stream);
 
 /* ---------------------------------------------------------------- sampling
  * TopKSampling.sample / TopPSampling.sample (src/rotor/generation.py:45-145) on the device: logits

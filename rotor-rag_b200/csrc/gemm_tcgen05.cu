@@ -26,8 +26,8 @@
 
 #include <cstdlib>
 
-#include "gemv_core.cuh"
 #include "model.cuh"
+#include "tc5.cuh"
 
 RB_TRACE_DEFINE(rotor_b200_trace_read_gemm5)
 
@@ -57,8 +57,6 @@ struct T5Cfg {
     static constexpr int THREADS = (DECODERS + 2) * 32;
     static constexpr int TILES_PER_WARP = ROWS / TILE_ROWS / DECODERS;  // row tiles each decoder warp handles
 };
-constexpr long long T5_SPIN_CYCLES = 400000000LL;  // about 0.2 s
-
 struct Tc5Params {
     const uint4* tiles;
     const int32_t* xsum;  // [ncols] sum of each token's int8 activations (removes the +1 of the weight codes)
@@ -85,94 +83,6 @@ struct Tc5Params {
     float* v_cache;
     float sq, sk, sv;
 };
-
-__device__ __forceinline__ bool t5_wait(uint32_t bar, uint32_t parity, volatile int* abort_flag, unsigned* status,
-                                        unsigned code) {
-    long long t0 = 0;
-    for (int it = 0;; ++it) {
-        uint32_t ok;
-        asm volatile(
-            "{ .reg .pred p; mbarrier.try_wait.parity.shared::cta.b64 p, [%1], %2; selp.u32 %0, 1, 0, p; }"
-            : "=r"(ok)
-            : "r"(bar), "r"(parity)
-            : "memory");
-        if (ok) return true;
-        if (*abort_flag) return false;
-        if (it == 0) t0 = clock64();
-        if (clock64() - t0 > T5_SPIN_CYCLES) {
-            *abort_flag = 1;
-            atomicExch(status, code);
-            return false;
-        }
-    }
-}
-
-// Shared-memory matrix descriptor, K-major, 128-byte swizzle: 8-row groups 1024 bytes apart.
-__device__ __forceinline__ uint64_t t5_desc(uint32_t smem_addr) {
-    return (uint64_t)((smem_addr >> 4) & 0x3fffu) | (1ull << 16) | ((uint64_t)(1024 >> 4) << 32) | (1ull << 46) |
-           (2ull << 61);
-}
-
-__device__ __forceinline__ void t5_ld32(uint32_t taddr, uint32_t (&v)[32]) {
-    asm volatile(
-        "tcgen05.ld.sync.aligned.32x32b.x32.b32 "
-        "{%0, %1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15, "
-        "%16, %17, %18, %19, %20, %21, %22, %23, %24, %25, %26, %27, %28, %29, %30, %31}, [%32];"
-        : "=r"(v[0]), "=r"(v[1]), "=r"(v[2]), "=r"(v[3]), "=r"(v[4]), "=r"(v[5]), "=r"(v[6]), "=r"(v[7]), "=r"(v[8]),
-          "=r"(v[9]), "=r"(v[10]), "=r"(v[11]), "=r"(v[12]), "=r"(v[13]), "=r"(v[14]), "=r"(v[15]), "=r"(v[16]),
-          "=r"(v[17]), "=r"(v[18]), "=r"(v[19]), "=r"(v[20]), "=r"(v[21]), "=r"(v[22]), "=r"(v[23]), "=r"(v[24]),
-          "=r"(v[25]), "=r"(v[26]), "=r"(v[27]), "=r"(v[28]), "=r"(v[29]), "=r"(v[30]), "=r"(v[31])
-        : "r"(taddr));
-}
-
-// Read-back store of a warp's 32 tokens x 32 values (lane = token after tcgen05.ld) as whole 128-byte
-// rows: through a per-warp shared-memory block (32 rows of 144 bytes: conflict-free both ways) so that
-// one store instruction covers four tokens' rows (four lines) instead of one 16-byte piece of 32
-// different lines.  dst0: address of token tok_base's first value; tokens at and beyond ntok are skipped.
-constexpr uint32_t T5_XPOSE_BYTES = 32 * 144;
-__device__ __forceinline__ void t5_store_rows(uint32_t stage, const uint32_t (&v)[32], void* dst0, size_t row_bytes,
-                                              int tok_base, int ntok, int lane) {
-#pragma unroll
-    for (int q = 0; q < 8; ++q)
-        asm volatile("st.shared.v4.u32 [%0], {%1, %2, %3, %4};" ::"r"(stage + (uint32_t)lane * 144u + 16u * q),
-                     "r"(v[4 * q]), "r"(v[4 * q + 1]), "r"(v[4 * q + 2]), "r"(v[4 * q + 3])
-                     : "memory");
-    __syncwarp();
-#pragma unroll
-    for (int i = 0; i < 8; ++i) {
-        const int tl = 4 * i + (lane >> 3);
-        uint4 w;
-        asm volatile("ld.shared.v4.u32 {%0, %1, %2, %3}, [%4];"
-                     : "=r"(w.x), "=r"(w.y), "=r"(w.z), "=r"(w.w)
-                     : "r"(stage + (uint32_t)tl * 144u + 16u * (lane & 7)));
-        if (tok_base + tl < ntok)
-            *reinterpret_cast<uint4*>(static_cast<unsigned char*>(dst0) + (size_t)tl * row_bytes + 16 * (lane & 7)) = w;
-    }
-    __syncwarp();  // the block is rewritten by the warp's next item
-}
-
-// The same with a destination per token: dst_of(tl) is the address of token tok_base + tl's 128 bytes
-// (null = skip).
-template <typename F>
-__device__ __forceinline__ void t5_store_rows_to(uint32_t stage, const uint32_t (&v)[32], int lane, F dst_of) {
-#pragma unroll
-    for (int q = 0; q < 8; ++q)
-        asm volatile("st.shared.v4.u32 [%0], {%1, %2, %3, %4};" ::"r"(stage + (uint32_t)lane * 144u + 16u * q),
-                     "r"(v[4 * q]), "r"(v[4 * q + 1]), "r"(v[4 * q + 2]), "r"(v[4 * q + 3])
-                     : "memory");
-    __syncwarp();
-#pragma unroll
-    for (int i = 0; i < 8; ++i) {
-        const int tl = 4 * i + (lane >> 3);
-        uint4 w;
-        asm volatile("ld.shared.v4.u32 {%0, %1, %2, %3}, [%4];"
-                     : "=r"(w.x), "=r"(w.y), "=r"(w.z), "=r"(w.w)
-                     : "r"(stage + (uint32_t)tl * 144u + 16u * (lane & 7)));
-        unsigned char* d = static_cast<unsigned char*>(dst_of(tl));
-        if (d) *reinterpret_cast<uint4*>(d + 16 * (lane & 7)) = w;
-    }
-    __syncwarp();
-}
 
 template <int ROWS, int T5_TOK = 256, bool GATED = false, bool QKV = false>
 __global__ void __launch_bounds__(T5Cfg<ROWS, T5_TOK>::THREADS, 1)

@@ -16,87 +16,10 @@
 #include <cstring>
 #include <new>
 
+#include "model_handle.cuh"
 #include "product_body.cuh"
 
 namespace rb {
-
-static inline size_t al256(size_t v) { return (v + 255) & ~(size_t)255; }
-
-// Scratch buffers and dimensions one block needs; carved from caller-owned device memory.
-struct Ctx {
-    int d, ff, n_heads, n_kv_heads, head_dim, dq, dkv;
-    int terms, ffn_act, causal, variant, max_seq;
-    float rope_theta, eps;
-    size_t kmax;  // widest padded BitLinear input
-    float* h;     // residual stream [rows][d]
-    float* h2;    // second copy: fused generation steps ping-pong between the two
-    float* hn;    // final-normed rows
-    float* qbuf;
-    float* attn;
-    int8_t* xq;
-    float* sx[2];
-    int32_t* xsum[2];
-    int32_t* accA;  // q/k/v and gate/up accumulators
-    int32_t* accB;  // o and down accumulators
-    int* d_pos;
-    float2* rope;        // cos/sin table, or null
-    float2* rope_buf;    // storage for it
-    __nv_bfloat16* kvsplit;  // prefill attention: hi / lo bf16 planes of one layer's K/V rows (or null)
-    size_t kvsplit_plane;
-    float* part_o;       // decode-attention partials
-    float* part_m;
-    float* part_l;
-    int nsplit;
-    int max_batch;
-    unsigned* counters;  // [8 + max_batch] zeroed words for last-CTA tails
-    // tensor parallel (tp_size > 1): communicator, whole FFN width, exchange buffers
-    void* tp;
-    int tp_size, ff_total;
-    float* stat[2];      // [rows] per-row statistics that cross ranks (sum of squares, absolute maximum)
-    float* gated;        // [rows][ff] this rank's slice of the gated FFN row
-    // float32 outputs of the fused generation step's products: q/k/v, o, gated, down
-    float* fy[4];
-};
-
-constexpr int FUSED_MAX_ROWS = 4;
-
-struct Model {
-    rotor_b200_model_config cfg;
-    rotor_b200_layer_weights* layers;
-    const __nv_bfloat16* embed;
-    const float* final_norm;
-    Ctx c;
-    float* part_val;
-    int* part_idx;
-    long long* cur_ids;
-    long long* tok_log;
-    int* d_step;
-    int* d_lens;                // [max_batch] prompt lengths of a ragged batch
-    const int32_t* last_of;     // host, during a ragged forward: tokens of each sequence (its last row is picked)
-    int max_log;
-    // host mirror of the generation state
-    int pos, step, batch;
-    cudaGraphExec_t graph;
-    int graph_batch;
-    unsigned long long graph_launches;  // kernels inside the captured step
-    // tensor parallel greedy pick: (value, global index) of every rank's best row
-    __nv_bfloat16* xsplit;  // LM head over more than four rows: hi / lo bf16 split of its input rows
-    float* pick_val;      // [rows]
-    long long* pick_idx;  // [rows]
-    unsigned char* pick_send;  // [rows] x 12 bytes
-    unsigned char* pick_recv;  // [tp][rows] x 12 bytes
-};
-
-struct Carve {
-    unsigned char* base;
-    size_t off;
-    template <typename T>
-    T* take(size_t count) {
-        T* p = base ? reinterpret_cast<T*>(base + off) : nullptr;
-        off += al256(count * sizeof(T));
-        return p;
-    }
-};
 
 static int max_planes(size_t out, size_t in) { return plan_gemv(out, in, 8).ksplit; }
 
@@ -248,12 +171,6 @@ __global__ void advance_kernel(const long long* cur, long long* log, int batch, 
     if (threadIdx.x < batch) pos[threadIdx.x] += 1;
     if (threadIdx.x == 0) *step = s + 1;
 }
-
-#define RB_TRY(expr)              \
-    do {                          \
-        int rc_ = (expr);         \
-        if (rc_) return rc_;      \
-    } while (0)
 
 // One BitLinear product into partial planes, activations taken from xq/xsum[xs].
 static int gemv(Ctx& c, const void* tiles, size_t out, size_t in, int ncols, int xs, int32_t* acc, AccView* view,
@@ -1000,6 +917,7 @@ static int run_step_fused_tp(Model& m, const long long* ids, int batch, long lon
 // ids: device [batch*seq]; the position is read from c.d_pos by the kernels.
 static int run_layers(Model& m, const long long* ids, int batch, int seq, int logits_mode, float* logits,
                       long long* next_ids, cudaStream_t st, bool advance = false) {
+    if (m.decoder) return run_decoder(m, ids, batch, seq, logits_mode, logits, next_ids, st, advance);
     Ctx& c = m.c;
     if (c.tp_size > 1) {
         if (!c.tp) return ROTOR_B200_ERR_ARG;  // rotor_b200_model_set_tp has not been called
@@ -1007,7 +925,7 @@ static int run_layers(Model& m, const long long* ids, int batch, int seq, int lo
             return run_step_fused_tp(m, ids, batch, next_ids, st, advance);
         return run_layers_tp(m, ids, batch, seq, logits_mode, logits, next_ids, st, advance);
     }
-    if (fused_step_ok(m, batch, seq) && (logits_mode != ROTOR_B200_LOGITS_NONE || next_ids))
+    if (!m.want && fused_step_ok(m, batch, seq) && (logits_mode != ROTOR_B200_LOGITS_NONE || next_ids))
         return run_step_fused(m, ids, batch, logits_mode, logits, next_ids, st, advance);
     const int rows = batch * seq, d = c.d;
     VecStageParams e = {};
@@ -1027,7 +945,15 @@ static int run_layers(Model& m, const long long* ids, int batch, int seq, int lo
     const bool all = logits_mode == ROTOR_B200_LOGITS_ALL;
     const float* x = c.hn;
     int lm_rows = rows;
-    if (!all && seq > 1) {
+    if (m.want) {
+        // compact the wanted rows: hn[want[i]] -> qbuf[i] (qbuf is free by now)
+        for (int i = 0; i < m.nwant; ++i)
+            RB_CUDA(cudaMemcpyAsync(c.qbuf + (size_t)i * d, c.hn + (size_t)m.want[i] * d, d * sizeof(float),
+                                    cudaMemcpyDeviceToDevice, st));
+        x = c.qbuf;
+        lm_rows = m.nwant;
+        if (!lm_rows) return ROTOR_B200_OK;
+    } else if (!all && seq > 1) {
         // compact the last rows: hn[b*seq + seq-1] -> qbuf[b] (qbuf is free by now)
         for (int b = 0; b < batch; ++b)
             RB_CUDA(cudaMemcpyAsync(c.qbuf + (size_t)b * d, c.hn + ((size_t)b * seq + (m.last_of ? m.last_of[b] : seq) - 1) * d, d * sizeof(float),
@@ -1044,7 +970,7 @@ static int run_layers(Model& m, const long long* ids, int batch, int seq, int lo
     lp.logits = logits_mode == ROTOR_B200_LOGITS_NONE ? nullptr : logits;
     lp.part_val = m.part_val;
     lp.part_idx = m.part_idx;
-    lp.argmax_out = (all && seq > 1) ? nullptr : next_ids;
+    lp.argmax_out = m.want || (all && seq > 1) ? nullptr : next_ids;
     lp.nparts = lmhead_parts();
     lp.tail_counter = c.counters + 3;
     if (advance) {
@@ -1122,6 +1048,7 @@ void rotor_b200_model_destroy(void* handle) {
     Model* m = (Model*)handle;
     if (!m) return;
     if (m->graph) cudaGraphExecDestroy(m->graph);
+    if (m->decoder) destroy_decoder(m->decoder);
     free(m->layers);
     delete m;
 }
@@ -1137,6 +1064,27 @@ int rotor_b200_model_forward(void* handle, const int64_t* ids, int batch, int se
     cudaStream_t st = as_stream(stream);
     set_pos_kernel<<<1, 256, 0, st>>>(m->c.d_pos, m->c.max_batch, past_len, nullptr);
     RB_TRY(run_layers(*m, (const long long*)ids, batch, seq, logits_mode, logits, (long long*)next_ids, st));
+    m->pos = past_len + seq;
+    return launch_status();
+}
+
+int rotor_b200_model_forward_rows(void* handle, const int64_t* ids, int batch, int seq, int past_len, const int32_t* rows,
+                                  int nrows, float* logits, void* stream) {
+    Model* m = (Model*)handle;
+    RB_REQUIRE(m && ids && batch > 0 && seq > 0 && past_len >= 0 && nrows >= 0 && m->c.tp_size <= 1);
+    RB_REQUIRE(batch <= m->cfg.max_batch && (long)batch * seq <= m->cfg.max_rows && past_len + seq <= m->cfg.max_seq);
+    RB_REQUIRE(nrows == 0 || (rows && logits && nrows <= batch * seq));
+    for (int i = 0; i < nrows; ++i) RB_REQUIRE(rows[i] >= 0 && rows[i] < batch * seq);
+    cudaStream_t st = as_stream(stream);
+    set_pos_kernel<<<1, 256, 0, st>>>(m->c.d_pos, m->c.max_batch, past_len, nullptr);
+    const int32_t none = 0;
+    m->want = nrows ? rows : &none;
+    m->nwant = nrows;
+    const int rc = run_layers(*m, (const long long*)ids, batch, seq, nrows ? ROTOR_B200_LOGITS_ALL : ROTOR_B200_LOGITS_NONE, logits,
+                              nullptr, st);
+    m->want = nullptr;
+    m->nwant = 0;
+    if (rc) return rc;
     m->pos = past_len + seq;
     return launch_status();
 }
@@ -1290,7 +1238,7 @@ int rotor_b200_model_forward_hidden(void* handle, const float* hidden_in, int ba
                                     int layer_begin, int layer_end, int apply_final_norm, float* hidden_out,
                                     void* stream) {
     Model* m = (Model*)handle;
-    RB_REQUIRE(m && hidden_in && hidden_out && batch > 0 && seq > 0 && past_len >= 0);
+    RB_REQUIRE(m && !m->decoder && hidden_in && hidden_out && batch > 0 && seq > 0 && past_len >= 0);
     RB_REQUIRE(batch <= m->cfg.max_batch && (long)batch * seq <= m->cfg.max_rows);
     RB_REQUIRE(past_len + seq <= m->cfg.max_seq);
     RB_REQUIRE(layer_begin >= 0 && layer_begin < layer_end && layer_end <= m->cfg.n_layers);

@@ -115,6 +115,38 @@ _SIGNATURES.update({
 })
 
 
+class DecoderConfig(C.Structure):
+    """rotor_b200_decoder_config"""
+    _fields_ = [("vocab_size", C.c_int32), ("width", C.c_int32), ("streams", C.c_int32), ("n_layers", C.c_int32),
+                ("n_runs", C.c_int32), ("f32", C.c_int32), ("eps", C.c_float),
+                ("max_batch", C.c_int32), ("max_seq", C.c_int32), ("max_rows", C.c_int32)]
+
+
+class DecoderLayer(C.Structure):
+    """rotor_b200_decoder_layer"""
+    _fields_ = [("heads", C.c_int32), ("kv_heads", C.c_int32), ("dim", C.c_int32), ("vdim", C.c_int32),
+                ("unit_qk", C.c_int32), ("chunk", C.c_int32), ("ff", C.c_int32), ("scale", _f), ("slopes", _p),
+                ("qkv", _p), ("o", _p), ("gate_up", _p), ("down", _p), ("norm1", _p), ("norm2", _p),
+                ("hc1_in", _p), ("hc1_out", _p), ("hc1_mix", _p), ("hc2_in", _p), ("hc2_out", _p), ("hc2_mix", _p)]
+
+
+class DecoderRun(C.Structure):
+    """rotor_b200_decoder_run"""
+    _fields_ = [("layer", C.c_int32), ("k_cache", _p), ("v_cache", _p)]
+
+
+_dcp, _dlp, _drp = C.POINTER(DecoderConfig), C.POINTER(DecoderLayer), C.POINTER(DecoderRun)
+
+_SIGNATURES.update({
+    "rotor_b200_model_forward_rows": (_i, [_p, _p, _i, _i, _i, _p, _i, _p, _p]),
+    "rotor_b200_decoder_workspace_bytes": (_sz, [_dcp, _dlp]),
+    "rotor_b200_decoder_create": (_i, [_dcp, _dlp, _drp, _p, _p, _p, _p, _sz, C.POINTER(_p)]),
+    "rotor_b200_stream_stage": (_i, [_p, _p, _i, _p, _p, _p, _p, _p, _p, _p, _f, _i, _i, _i, _p, _i, _p]),
+    "rotor_b200_dense_linear": (_i, [_p, _i, _i, _p, _i, _i, _i, _p, _p, _p]),
+    "rotor_b200_bias_attention": (_i, [_dlp, _f, _i, _p, _i, _i, _p, _i, _p, _p, _p, _i, _p, _p]),
+})
+
+
 def _declare(signatures):
     for name, (res, args) in signatures.items():
         fn = getattr(lib, name)  # AttributeError here = header and library out of step
