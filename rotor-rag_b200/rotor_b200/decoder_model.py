@@ -116,8 +116,7 @@ class _DecoderHandle:
 
     def __del__(self):
         h, self.h = getattr(self, "h", None), None
-        if h:
-            abi.require_cuda().cuda.synchronize()
+        if h and lib is not None:   # (module globals are gone at interpreter exit)
             lib.rotor_b200_model_destroy(h)
 
 
