@@ -184,25 +184,6 @@ __global__ void dequant_kernel(const int32_t* __restrict__ acc, const float* __r
     }
 }
 
-// Device status word shared by every launch of the library on one device (one word per device).
-static PerDevice<unsigned*> g_status_words;
-static int ensure_status() {
-    unsigned*& w = g_status_words.here();
-    if (w) return ROTOR_B200_OK;
-    RB_CUDA(cudaMalloc(&w, sizeof(unsigned)));
-    RB_CUDA(cudaMemset(w, 0, sizeof(unsigned)));
-    return ROTOR_B200_OK;
-}
-
-__global__ void empty_kernel() {
-    pdl_wait();
-    pdl_trigger();
-}
-
-int g_use_pdl = 1;  // programmatic dependent launch for the kernels that call pdl_wait()
-
-unsigned* library_status_word() { return ensure_status() ? nullptr : g_status_words.here(); }
-
 template <int WARPS, int UMAX, bool USE_MMA, int NCOL>
 static int launch_acc(const AccParams& p, int nrt, int ksplit, cudaStream_t st) {
     auto kern = bitlinear_acc_kernel<WARPS, UMAX, USE_MMA, NCOL>;
@@ -269,7 +250,7 @@ static int configure_one() {
 
 // Done once, outside any stream capture: status word and the shared-memory opt-ins.
 int configure_gemv_kernels() {
-    int rc = ensure_status();
+    int rc = (library_status_word() ? ROTOR_B200_OK : ROTOR_B200_ERR_CUDA);
     if (rc) return rc;
     if ((rc = configure_one<true, 1>())) return rc;
     if ((rc = configure_one<false, 1>())) return rc;
@@ -299,7 +280,7 @@ GemvPlan plan_gemv(size_t out, size_t in, int ncols) {
 
 int launch_gemv_planes(const void* tiles, size_t out, size_t in, const int8_t* xq, const int32_t* xsum, int ncols,
                        int32_t* acc, size_t plane_stride, const GemvPlan& plan, int variant, cudaStream_t st) {
-    int rc = ensure_status();
+    int rc = (library_status_word() ? ROTOR_B200_OK : ROTOR_B200_ERR_CUDA);
     if (rc) return rc;
     if (ncols >= GEMM_MIN_COLS && variant == ROTOR_B200_VARIANT_AUTO) {
         // compute-bound regime: the tiled GEMM writes complete sums into plane 0 (callers use one plane)
@@ -316,7 +297,7 @@ int launch_gemv_planes(const void* tiles, size_t out, size_t in, const int8_t* x
         p.xq = xq + (size_t)c0 * kpad;
         p.xsum = xsum + c0;
         p.acc = acc + (size_t)c0 * out;
-        p.status = g_status_words.here();
+        p.status = library_status_word();
         p.out = (int)out;
         p.nkt = nkt;
         p.kt_per_split = plan.kt_per_split;
@@ -343,7 +324,7 @@ int rotor_b200_bitlinear_acc(const void* tiles, size_t out, size_t in, const int
     RB_REQUIRE(out < (1u << 30) && in < (1u << 30));
     RB_REQUIRE(((uintptr_t)tiles & 15) == 0 && ((uintptr_t)xq & 15) == 0);
     RB_REQUIRE(variant >= ROTOR_B200_VARIANT_AUTO && variant <= ROTOR_B200_VARIANT_MMA);
-    int rc = ensure_status();
+    int rc = (library_status_word() ? ROTOR_B200_OK : ROTOR_B200_ERR_CUDA);
     if (rc) return rc;
     cudaStream_t st = as_stream(stream);
     const int nkt = (int)(kpad_of(in) / TILE_K), nrt = (int)(opad_of(out) / TILE_ROWS);
@@ -367,7 +348,7 @@ int rotor_b200_bitlinear_acc(const void* tiles, size_t out, size_t in, const int
         p.xq = xq + c0 * kpad;
         p.xsum = xsum + c0;
         p.acc = acc + c0 * out;
-        p.status = g_status_words.here();
+        p.status = library_status_word();
         p.out = (int)out;
         p.nkt = nkt;
         p.kt_per_split = (nkt + ksplit - 1) / ksplit;
@@ -457,6 +438,7 @@ static int static_scratch_address(unsigned char** out) {
         void* p = nullptr;
         RB_CUDA(cudaGetSymbolAddress(&p, g_static_scratch));
         addr = static_cast<unsigned char*>(p);
+        g_extra_status.v[dev] = reinterpret_cast<unsigned*>(addr);  // (its status word is at the start)
     }
     *out = addr;
     return ROTOR_B200_OK;
@@ -551,43 +533,6 @@ int rotor_b200_ternary_matmul_host(const void* tiles, const float* scales_host, 
     if (rc) return rc;
     RB_CUDA(cudaMemcpy(y_host, dy, out * 4, cudaMemcpyDeviceToHost));
     return ROTOR_B200_OK;
-}
-
-/* Measurement aid: one launch of a kernel that does nothing, with the same launch attributes
- * (programmatic dependent launch when enabled) as the kernels of the decode chain.  A chain of
- * these in a CUDA graph gives the floor that any chain of dependent launches pays per launch. */
-int rotor_b200_launch_empty(void* stream) {
-    cudaLaunchConfig_t cfg = {};
-    cfg.gridDim = dim3(148);
-    cfg.blockDim = dim3(128);
-    cfg.stream = as_stream(stream);
-    cudaLaunchAttribute attr[1];
-    attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
-    attr[0].val.programmaticStreamSerializationAllowed = 1;
-    cfg.attrs = attr;
-    cfg.numAttrs = g_use_pdl ? 1 : 0;
-    if (cudaLaunchKernelEx(&cfg, rb::empty_kernel) != cudaSuccess) {
-        ++g_launch_count;
-        return ROTOR_B200_ERR_CUDA;
-    }
-    return launch_status();
-}
-
-/* Reads and clears the status words of the current device that bounded waits write to: the
- * library's own word and the one at the start of the fixed scratch array of
- * rotor_b200_bitlinear_forward_static (once that entry point has run on this device).  Allocates
- * nothing. */
-int rotor_b200_device_status(void) {
-    unsigned v = 0, vs = 0;
-    if (unsigned* w = g_status_words.here()) {
-        RB_CUDA(cudaMemcpy(&v, w, sizeof(v), cudaMemcpyDeviceToHost));
-        if (v) RB_CUDA(cudaMemset(w, 0, sizeof(v)));
-    }
-    if (unsigned char* a = g_static_addr.here()) {
-        RB_CUDA(cudaMemcpy(&vs, a, sizeof(vs), cudaMemcpyDeviceToHost));
-        if (vs) RB_CUDA(cudaMemset(a, 0, sizeof(vs)));
-    }
-    return (int)(v ? v : vs);
 }
 
 }  // extern "C"

@@ -1,7 +1,7 @@
 // Driver of layer-described decoders: a list of layer runs (a layer may run several times in a row with
 // the same weights, each run with its own cache), residual streams with hyper-connections, bias / chunk
 // attention, gated feed-forward, an output head of its own.  It sits behind the same model handle as the
-// ternary model: position state, generation loop, token log and captured graph are model.cu's.
+// ternary model: position state, generation loop, token log and captured graph are handle.cu's.
 //
 // Launch sequence of a forward, per layer run
 //   many rows:  stage (streams, norm) -> q/k/v product [-> head finish] -> attention -> o product
@@ -115,9 +115,7 @@ static void carve_decoder(Model& m, DecoderStack& d, const rotor_b200_decoder_la
     *total = cv.off;
 }
 
-void destroy_decoder(DecoderStack* d) { delete d; }
-
-int run_decoder(Model& m, const long long* ids, int batch, int seq, int logits_mode, float* logits, long long* next_ids,
+static int run_decoder(Model& m, const long long* ids, int batch, int seq, int logits_mode, float* logits, long long* next_ids,
                 cudaStream_t st, bool advance) {
     DecoderStack& d = *m.decoder;
     const rotor_b200_decoder_config& c = d.cfg;
@@ -279,6 +277,9 @@ int run_decoder(Model& m, const long long* ids, int batch, int seq, int logits_m
     return launch_lmhead(lp, lm_rows, st);
 }
 
+static void destroy_decoder(Model& m) { delete m.decoder; }
+static const ModelFamily DECODER_FAMILY = {run_decoder, destroy_decoder};
+
 }  // namespace rb
 
 using namespace rb;
@@ -316,6 +317,7 @@ int rotor_b200_decoder_create(const rotor_b200_decoder_config* cfg, const rotor_
         return ROTOR_B200_ERR_ARG;
     }
     memset(m, 0, sizeof(*m));
+    m->family = &DECODER_FAMILY;
     m->decoder = d;
     m->no_fused = getenv("ROTOR_B200_NO_FUSED_STEP") != nullptr;
     d->cfg = *cfg;

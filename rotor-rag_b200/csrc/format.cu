@@ -9,8 +9,6 @@
 
 namespace rb {
 
-unsigned long long g_launch_count = 0;
-
 __global__ void encode_kernel(const int8_t* __restrict__ w, size_t n, uint8_t* __restrict__ plus,
                               uint8_t* __restrict__ minus) {
     for (size_t i = blockIdx.x * (size_t)blockDim.x + threadIdx.x; i < n; i += (size_t)gridDim.x * blockDim.x) {
@@ -160,23 +158,6 @@ static inline unsigned grid_for(size_t n, unsigned block = 256) {
 using namespace rb;
 
 extern "C" {
-
-int rotor_b200_version(void) { return 100; }
-
-unsigned long long rotor_b200_launch_count(void) { return g_launch_count; }
-
-const char* rotor_b200_status_string(int status) {
-    switch (status) {
-        case ROTOR_B200_OK: return "ok";
-        case ROTOR_B200_ERR_ARG: return "invalid argument";
-        case ROTOR_B200_ERR_CUDA: return "CUDA error";
-        case ROTOR_B200_ERR_SHAPE: return "unsupported shape";
-        case ROTOR_B200_ERR_WORKSPACE: return "workspace too small";
-        case ROTOR_B200_ERR_TIMEOUT: return "device-side wait timed out";
-        case ROTOR_B200_ERR_TOO_LARGE: return "problem exceeds the library's built-in scratch array";
-        default: return "unknown status";
-    }
-}
 
 int rotor_b200_encode(const int8_t* w, size_t n, uint8_t* plus, uint8_t* minus, void* stream) {
     if (n == 0) return ROTOR_B200_OK;

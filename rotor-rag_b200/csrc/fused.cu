@@ -46,16 +46,6 @@ __global__ void __launch_bounds__(FG_THREADS, DEEP ? 1 : 2) fused_gemv_kernel(co
     RB_TRACE_COMMIT(tr, p.st.mode * 10 + p.halves);
 }
 
-static PerDevice<int> g_sm_counts;
-static int sm_count() {
-    int& n = g_sm_counts.here();
-    if (!n) {
-        if (cudaDeviceGetAttribute(&n, cudaDevAttrMultiProcessorCount, current_device()) != cudaSuccess || n <= 0)
-            n = 148;
-    }
-    return n;
-}
-
 template <bool USE_MMA, int NCOL, bool WIDE, bool DEEP, bool TP>
 static int launch_fused_tp(const FusedGemvParams& p, int grid, cudaStream_t st) {
     static PerDevice<bool> once;  // each variant raises its own shared-memory limit once per device
@@ -105,7 +95,7 @@ int configure_fused_gemv() {
     RB_CUDA(cudaFuncSetAttribute(fused_gemv_kernel<false, 1, true, true, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, big));
     RB_CUDA(cudaFuncSetAttribute(fused_gemv_kernel<false, 2, true, true, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, big));
     RB_CUDA(cudaFuncSetAttribute(fused_gemv_kernel<true, 1, true, true, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, big));
-    sm_count();
+    fused_sm_count();
     return ROTOR_B200_OK;
 }
 
@@ -121,7 +111,7 @@ bool fused_gemv_supported(size_t out, size_t in, int rows, int terms, int halves
     p.nkt = (int)(kpad_of(in) / TILE_K);
     p.halves = halves;
     const int units = (int)(opad_of(out) / TILE_ROWS);
-    p.upc = (units + sm_count() - 1) / sm_count();
+    p.upc = (units + fused_sm_count() - 1) / fused_sm_count();
     p.st.mode = merge_weights ? LM_ATTN : LM_ADD;
     p.st.n_heads = merge_weights;
     p.st.nsplit = 1;
@@ -131,7 +121,7 @@ bool fused_gemv_supported(size_t out, size_t in, int rows, int terms, int halves
 int launch_fused_gemv(const void* tiles, size_t out, size_t in, int halves, int rows, const LeanStage& stage, float* y,
                       const float* scale, int seg1, int seg2, int ffn_act, cudaStream_t st, const FusedTpExtra* tp) {
     FusedGemvParams p;
-    int grid = sm_count();
+    int grid = fused_sm_count();
     int rc = make_fused_params(p, tiles, out, in, halves, rows, stage, y, scale, seg1, seg2, ffn_act, grid);
     if (rc) return rc;
     if (tp) {
@@ -159,8 +149,6 @@ int launch_fused_gemv(const void* tiles, size_t out, size_t in, int halves, int 
     return launch_fused<true, 1, false, false>(p, grid, st);
 }
 
-int fused_sm_count() { return sm_count(); }
-
 // Stand-alone integer product through the staged kernel: the matrix is small enough for every
 // CTA's share of the tiles to sit in shared memory, and the activations are quantised already.
 bool staged_acc_supported(size_t out, size_t in, int ncols, int variant) {
@@ -171,7 +159,7 @@ bool staged_acc_supported(size_t out, size_t in, int ncols, int variant) {
     p.nkt = (int)(kpad_of(in) / TILE_K);
     p.halves = 1;
     p.units = (int)(opad_of(out) / TILE_ROWS);
-    const int grid = sm_count() < p.units ? sm_count() : p.units;
+    const int grid = fused_sm_count() < p.units ? fused_sm_count() : p.units;
     p.upc = (p.units + grid - 1) / grid;
     p.st.mode = LM_PLAIN;
     p.st.n = (int)in;
@@ -188,7 +176,7 @@ int launch_staged_acc(const void* tiles, size_t out, size_t in, const int8_t* xq
     stage.terms = 1;
     stage.kpad = (int)kpad_of(in);
     FusedGemvParams p;
-    int grid = sm_count();
+    int grid = fused_sm_count();
     const float one[3] = {1.f, 1.f, 1.f};
     int rc = make_fused_params(p, tiles, out, in, 1, ncols, stage, nullptr, one, (int)out, (int)out, 0, grid);
     if (rc) return rc;

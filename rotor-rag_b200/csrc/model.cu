@@ -149,29 +149,6 @@ static int derive(Model& m) {
     return ROTOR_B200_OK;
 }
 
-// Cached length of every sequence: one value for all, or lens[b] when given.
-__global__ void set_pos_kernel(int* pos, int n, int v, const int* lens) {
-    for (int i = threadIdx.x; i < n; i += blockDim.x) pos[i] = lens ? lens[i] : v;
-}
-
-__global__ void begin_kernel(long long* cur, const long long* first, int batch, int* pos, int past, const int* lens,
-                             int* step) {
-    if (threadIdx.x < batch) {
-        cur[threadIdx.x] = first[threadIdx.x];
-        pos[threadIdx.x] = lens ? lens[threadIdx.x] : past;
-    }
-    if (threadIdx.x == 0) *step = 0;
-}
-
-// After a generation step: log the picked tokens and move the position on.
-__global__ void advance_kernel(const long long* cur, long long* log, int batch, int max_log, int* pos, int* step) {
-    const int s = *step;
-    if (threadIdx.x < batch && s < max_log) log[(size_t)s * batch + threadIdx.x] = cur[threadIdx.x];
-    __syncthreads();
-    if (threadIdx.x < batch) pos[threadIdx.x] += 1;
-    if (threadIdx.x == 0) *step = s + 1;
-}
-
 // One BitLinear product into partial planes, activations taken from xq/xsum[xs].
 static int gemv(Ctx& c, const void* tiles, size_t out, size_t in, int ncols, int xs, int32_t* acc, AccView* view,
                 cudaStream_t st) {
@@ -779,8 +756,7 @@ static int run_layers_tp(Model& m, const long long* ids, int batch, int seq, int
         RB_TRY(launch_status());
     }
     if (advance) {
-        advance_kernel<<<1, 1024, 0, st>>>(next_ids, m.tok_log, batch, m.max_log, c.d_pos, m.d_step);
-        RB_TRY(launch_status());
+        RB_TRY(launch_advance(m, next_ids, batch, st));
     }
     return ROTOR_B200_OK;
 }
@@ -907,8 +883,7 @@ static int run_step_fused_tp(Model& m, const long long* ids, int batch, long lon
     final_pick_kernel<<<(batch + 127) / 128, 128, 0, st>>>(m.pick_recv, c.tp_size, batch, next_ids);
     RB_TRY(launch_status());
     if (advance) {
-        advance_kernel<<<1, 1024, 0, st>>>(next_ids, m.tok_log, batch, m.max_log, c.d_pos, m.d_step);
-        RB_TRY(launch_status());
+        RB_TRY(launch_advance(m, next_ids, batch, st));
     }
     return tp_step_end(c.tp, xi, st);
 }
@@ -916,8 +891,7 @@ static int run_step_fused_tp(Model& m, const long long* ids, int batch, long lon
 
 // ids: device [batch*seq]; the position is read from c.d_pos by the kernels.
 static int run_layers(Model& m, const long long* ids, int batch, int seq, int logits_mode, float* logits,
-                      long long* next_ids, cudaStream_t st, bool advance = false) {
-    if (m.decoder) return run_decoder(m, ids, batch, seq, logits_mode, logits, next_ids, st, advance);
+                      long long* next_ids, cudaStream_t st, bool advance) {
     Ctx& c = m.c;
     if (c.tp_size > 1) {
         if (!c.tp) return ROTOR_B200_ERR_ARG;  // rotor_b200_model_set_tp has not been called
@@ -982,6 +956,9 @@ static int run_layers(Model& m, const long long* ids, int batch, int seq, int lo
     return launch_lmhead(lp, lm_rows, st);
 }
 
+static void destroy_ternary(Model& m) { free(m.layers); }
+static const ModelFamily TERNARY_FAMILY = {run_layers, destroy_ternary};
+
 }  // namespace rb
 
 using namespace rb;
@@ -1007,6 +984,7 @@ int rotor_b200_model_create(const rotor_b200_model_config* cfg, const rotor_b200
     Model* m = new (std::nothrow) Model;
     if (!m) return ROTOR_B200_ERR_ARG;
     memset(m, 0, sizeof(*m));
+    m->family = &TERNARY_FAMILY;
     m->cfg = *cfg;
     int rc = derive(*m);
     if (rc) {
@@ -1044,168 +1022,6 @@ int rotor_b200_model_create(const rotor_b200_model_config* cfg, const rotor_b200
     return ROTOR_B200_OK;
 }
 
-void rotor_b200_model_destroy(void* handle) {
-    Model* m = (Model*)handle;
-    if (!m) return;
-    if (m->graph) cudaGraphExecDestroy(m->graph);
-    if (m->decoder) destroy_decoder(m->decoder);
-    free(m->layers);
-    delete m;
-}
-
-int rotor_b200_model_forward(void* handle, const int64_t* ids, int batch, int seq, int past_len, int logits_mode,
-                             float* logits, int64_t* next_ids, void* stream) {
-    Model* m = (Model*)handle;
-    RB_REQUIRE(m && ids && batch > 0 && seq > 0 && past_len >= 0);
-    RB_REQUIRE(batch <= m->cfg.max_batch && (long)batch * seq <= m->cfg.max_rows);
-    RB_REQUIRE(past_len + seq <= m->cfg.max_seq);
-    RB_REQUIRE(logits_mode >= ROTOR_B200_LOGITS_NONE && logits_mode <= ROTOR_B200_LOGITS_ALL);
-    RB_REQUIRE(logits_mode == ROTOR_B200_LOGITS_NONE || logits);
-    cudaStream_t st = as_stream(stream);
-    set_pos_kernel<<<1, 256, 0, st>>>(m->c.d_pos, m->c.max_batch, past_len, nullptr);
-    RB_TRY(run_layers(*m, (const long long*)ids, batch, seq, logits_mode, logits, (long long*)next_ids, st));
-    m->pos = past_len + seq;
-    return launch_status();
-}
-
-int rotor_b200_model_forward_rows(void* handle, const int64_t* ids, int batch, int seq, int past_len, const int32_t* rows,
-                                  int nrows, float* logits, void* stream) {
-    Model* m = (Model*)handle;
-    RB_REQUIRE(m && ids && batch > 0 && seq > 0 && past_len >= 0 && nrows >= 0 && m->c.tp_size <= 1);
-    RB_REQUIRE(batch <= m->cfg.max_batch && (long)batch * seq <= m->cfg.max_rows && past_len + seq <= m->cfg.max_seq);
-    RB_REQUIRE(nrows == 0 || (rows && logits && nrows <= batch * seq));
-    for (int i = 0; i < nrows; ++i) RB_REQUIRE(rows[i] >= 0 && rows[i] < batch * seq);
-    cudaStream_t st = as_stream(stream);
-    set_pos_kernel<<<1, 256, 0, st>>>(m->c.d_pos, m->c.max_batch, past_len, nullptr);
-    const int32_t none = 0;
-    m->want = nrows ? rows : &none;
-    m->nwant = nrows;
-    const int rc = run_layers(*m, (const long long*)ids, batch, seq, nrows ? ROTOR_B200_LOGITS_ALL : ROTOR_B200_LOGITS_NONE, logits,
-                              nullptr, st);
-    m->want = nullptr;
-    m->nwant = 0;
-    if (rc) return rc;
-    m->pos = past_len + seq;
-    return launch_status();
-}
-
-int rotor_b200_model_decode_begin(void* handle, const int64_t* first_ids, int batch, int past_len, void* stream) {
-    Model* m = (Model*)handle;
-    RB_REQUIRE(m && first_ids && batch > 0 && batch <= m->cfg.max_batch && batch <= 1024);
-    RB_REQUIRE(past_len >= 0 && past_len < m->cfg.max_seq);
-    begin_kernel<<<1, 1024, 0, as_stream(stream)>>>(m->cur_ids, (const long long*)first_ids, batch, m->c.d_pos,
-                                                    past_len, nullptr, m->d_step);
-    m->pos = past_len;
-    m->step = 0;
-    m->batch = batch;
-    return launch_status();
-}
-
-/* Prefill of a ragged batch: `ids` holds `batch` prompts right-padded to `seq` tokens (any valid
- * id as padding), lens[b] (host) the true length of prompt b, 1 <= lens[b] <= seq.  Causal
- * models only: a row then never sees the padding behind it, so every position below lens[b]
- * is what a batch-of-one forward of prompt b alone gives.  Logits / picks are taken at each
- * prompt's own last token (logits_mode NONE or LAST).  Cache positions lens[b].. hold padding
- * products; rotor_b200_model_decode_begin_ragged makes the next steps overwrite them in order. */
-int rotor_b200_model_forward_ragged(void* handle, const int64_t* ids, int batch, int seq, const int32_t* lens,
-                                    int logits_mode, float* logits, int64_t* next_ids, void* stream) {
-    Model* m = (Model*)handle;
-    RB_REQUIRE(m && ids && lens && batch > 0 && seq > 0);
-    RB_REQUIRE(m->cfg.causal && m->c.tp_size <= 1);
-    RB_REQUIRE(batch <= m->cfg.max_batch && (long)batch * seq <= m->cfg.max_rows && seq <= m->cfg.max_seq);
-    RB_REQUIRE(logits_mode == ROTOR_B200_LOGITS_NONE || (logits_mode == ROTOR_B200_LOGITS_LAST && logits));
-    for (int b = 0; b < batch; ++b) RB_REQUIRE(lens[b] >= 1 && lens[b] <= seq);
-    cudaStream_t st = as_stream(stream);
-    set_pos_kernel<<<1, 256, 0, st>>>(m->c.d_pos, m->c.max_batch, 0, nullptr);
-    m->last_of = lens;
-    const int rc = run_layers(*m, (const long long*)ids, batch, seq, logits_mode, logits, (long long*)next_ids, st);
-    m->last_of = nullptr;
-    if (rc) return rc;
-    m->pos = seq;
-    return launch_status();
-}
-
-/* rotor_b200_model_decode_begin for sequences of different cached lengths (host lens[b], after
- * rotor_b200_model_forward_ragged): sequence b appends at position lens[b] + step and attends
- * to its own lens[b] + step + 1 keys. */
-int rotor_b200_model_decode_begin_ragged(void* handle, const int64_t* first_ids, int batch, const int32_t* lens,
-                                         void* stream) {
-    Model* m = (Model*)handle;
-    RB_REQUIRE(m && first_ids && lens && batch > 0 && batch <= m->cfg.max_batch && batch <= 1024);
-    int longest = 0;
-    for (int b = 0; b < batch; ++b) {
-        RB_REQUIRE(lens[b] >= 0 && lens[b] < m->cfg.max_seq);
-        longest = lens[b] > longest ? lens[b] : longest;
-    }
-    cudaStream_t st = as_stream(stream);
-    RB_CUDA(cudaMemcpyAsync(m->d_lens, lens, (size_t)batch * sizeof(int), cudaMemcpyHostToDevice, st));
-    begin_kernel<<<1, 1024, 0, st>>>(m->cur_ids, (const long long*)first_ids, batch, m->c.d_pos, 0, m->d_lens,
-                                     m->d_step);
-    RB_CUDA(cudaStreamSynchronize(st));  // `lens` may be pageable host memory the caller reuses
-    m->pos = longest;  // capacity checks follow the longest sequence
-    m->step = 0;
-    m->batch = batch;
-    return launch_status();
-}
-
-static int one_step(Model& m, cudaStream_t st) {
-    if (m.c.tp_size > 1)
-        return run_layers(m, m.cur_ids, m.batch, 1, ROTOR_B200_LOGITS_NONE, nullptr, m.cur_ids, st, true);
-    if (m.batch <= 4)  // pick, token log and position advance ride in the LM head's last CTA
-        return run_layers(m, m.cur_ids, m.batch, 1, ROTOR_B200_LOGITS_NONE, nullptr, m.cur_ids, st, true);
-    RB_TRY(run_layers(m, m.cur_ids, m.batch, 1, ROTOR_B200_LOGITS_NONE, nullptr, m.cur_ids, st));
-    advance_kernel<<<1, 1024, 0, st>>>(m.cur_ids, m.tok_log, m.batch, m.max_log, m.c.d_pos, m.d_step);
-    return launch_status();
-}
-
-int rotor_b200_model_decode_steps(void* handle, int nsteps, int use_graph, void* stream) {
-    Model* m = (Model*)handle;
-    RB_REQUIRE(m && nsteps > 0 && m->batch > 0);
-    RB_REQUIRE(m->pos + nsteps <= m->cfg.max_seq && m->step + nsteps <= m->max_log);
-    cudaStream_t st = as_stream(stream);
-    if (!use_graph) {
-        for (int i = 0; i < nsteps; ++i) RB_TRY(one_step(*m, st));
-    } else {
-        if (m->graph && (m->graph_batch != m->batch)) {
-            cudaGraphExecDestroy(m->graph);
-            m->graph = nullptr;
-        }
-        if (!m->graph) {
-            RB_REQUIRE(st != nullptr);  // the legacy default stream cannot be captured
-            cudaGraph_t g = nullptr;
-            RB_CUDA(cudaStreamBeginCapture(st, cudaStreamCaptureModeThreadLocal));
-            const unsigned long long before = g_launch_count;
-            int rc = one_step(*m, st);
-            m->graph_launches = g_launch_count - before;
-            g_launch_count = before;  // captured, not run
-            cudaError_t e = cudaStreamEndCapture(st, &g);
-            if (rc || e != cudaSuccess) {
-                if (g) cudaGraphDestroy(g);
-                return rc ? rc : ROTOR_B200_ERR_CUDA;
-            }
-            e = cudaGraphInstantiate(&m->graph, g, 0);
-            cudaGraphDestroy(g);
-            if (e != cudaSuccess) return ROTOR_B200_ERR_CUDA;
-            m->graph_batch = m->batch;
-        }
-        for (int i = 0; i < nsteps; ++i) RB_CUDA(cudaGraphLaunch(m->graph, st));
-        g_launch_count += m->graph_launches * (unsigned long long)nsteps;
-    }
-    m->pos += nsteps;
-    m->step += nsteps;
-    return ROTOR_B200_OK;
-}
-
-int rotor_b200_model_read_tokens(void* handle, int first_step, int count, int64_t* tokens_host, void* stream) {
-    Model* m = (Model*)handle;
-    RB_REQUIRE(m && tokens_host && first_step >= 0 && count > 0 && first_step + count <= m->step);
-    cudaStream_t st = as_stream(stream);
-    RB_CUDA(cudaMemcpyAsync(tokens_host, m->tok_log + (size_t)first_step * m->batch,
-                            (size_t)count * m->batch * sizeof(int64_t), cudaMemcpyDeviceToHost, st));
-    RB_CUDA(cudaStreamSynchronize(st));
-    return ROTOR_B200_OK;
-}
-
 /* Attaches the tensor-parallel communicator (made by rotor_b200_tp_init) to a model created with
  * tp_size > 1.  The handle's rank must match the configuration's tp_rank. */
 int rotor_b200_model_set_tp(void* handle, void* comm) {
@@ -1216,20 +1032,6 @@ int rotor_b200_model_set_tp(void* handle, void* comm) {
     return ROTOR_B200_OK;
 }
 
-/* Programmatic dependent launch for the kernels of the decode chain: 1 lets each kernel start
- * (and prefetch its weight tiles) while its predecessor drains.  Applies to later launches and
- * to graphs captured afterwards.  Returns the previous setting. */
-int rotor_b200_set_pdl(int enable) {
-    const int old = g_use_pdl;
-    g_use_pdl = enable ? 1 : 0;
-    return old;
-}
-
-int rotor_b200_model_position(void* handle) {
-    Model* m = (Model*)handle;
-    return m ? m->pos : -1;
-}
-
 /* Runs blocks [layer_begin, layer_end) of the model on caller-provided hidden rows
  * (float32 [batch*seq][d_model], device).  With apply_final_norm the model's final norm is
  * applied to the result (BitNetModel.forward(return_logits=False), bitnet_model.py:231-243);
@@ -1238,14 +1040,14 @@ int rotor_b200_model_forward_hidden(void* handle, const float* hidden_in, int ba
                                     int layer_begin, int layer_end, int apply_final_norm, float* hidden_out,
                                     void* stream) {
     Model* m = (Model*)handle;
-    RB_REQUIRE(m && !m->decoder && hidden_in && hidden_out && batch > 0 && seq > 0 && past_len >= 0);
+    RB_REQUIRE(m && m->family == &TERNARY_FAMILY && hidden_in && hidden_out && batch > 0 && seq > 0 && past_len >= 0);
     RB_REQUIRE(batch <= m->cfg.max_batch && (long)batch * seq <= m->cfg.max_rows);
     RB_REQUIRE(past_len + seq <= m->cfg.max_seq);
     RB_REQUIRE(layer_begin >= 0 && layer_begin < layer_end && layer_end <= m->cfg.n_layers);
     cudaStream_t st = as_stream(stream);
     Ctx& c = m->c;
     const int rows = batch * seq;
-    set_pos_kernel<<<1, 256, 0, st>>>(c.d_pos, c.max_batch, past_len, nullptr);
+    RB_TRY(launch_set_pos(c.d_pos, c.max_batch, past_len, nullptr, st));
     RB_CUDA(cudaMemcpyAsync(c.h, hidden_in, (size_t)rows * c.d * sizeof(float), cudaMemcpyDeviceToDevice, st));
     VecStageParams e = {};
     e.mode = VS_PLAIN;
@@ -1388,7 +1190,7 @@ int rotor_b200_attention_forward(const rotor_b200_model_config* cfg, const rotor
     Ctx c;
     cudaStream_t st = as_stream(stream);
     RB_TRY(block_ctx(c, cfg, rows, workspace, workspace_bytes, st));
-    set_pos_kernel<<<1, 256, 0, st>>>(c.d_pos, c.max_batch, past_len, nullptr);
+    RB_TRY(launch_set_pos(c.d_pos, c.max_batch, past_len, nullptr, st));
     VecStageParams e = {};
     e.mode = VS_PLAIN;
     e.n = c.d;

@@ -227,6 +227,8 @@ int launch_lmhead(const LmHeadParams& p, int rows, cudaStream_t st);
 int lmhead_parts();
 
 unsigned* library_status_word();
+// a second status word of the current device that rotor_b200_device_status() reads, once one exists
+extern PerDevice<unsigned*> g_extra_status;
 
 // Tensor-parallel collectives (tp.cu); `comm` is the handle made by rotor_b200_tp_init.
 int tp_rank(void* comm);

@@ -1,6 +1,6 @@
 // State behind a model handle, shared by the drivers of the model families (model.cu: the ternary
 // model; decoder.cu: decoders described layer by layer).  The generation loop, its token log and its
-// captured graph work on this state whatever the family.
+// captured graph (handle.cu) work on this state whatever the family.
 #pragma once
 #include "model.cuh"
 
@@ -14,7 +14,17 @@ namespace rb {
 
 inline size_t al256(size_t v) { return (v + 255) & ~(size_t)255; }
 
+struct Model;
 struct DecoderStack;
+
+// What a family supplies.  forward: one forward over ids (device [batch * seq]); cached lengths are read
+// from m.c.d_pos; logits of the last positions, of all, or of the rows m.want; with `advance` the call is a
+// generation step that also logs its picks and moves the positions on.
+struct ModelFamily {
+    int (*forward)(Model& m, const long long* ids, int batch, int seq, int logits_mode, float* logits,
+                   long long* next_ids, cudaStream_t st, bool advance);
+    void (*destroy)(Model& m);
+};
 
 // Scratch buffers and dimensions one block needs; carved from caller-owned device memory.
 struct Ctx {
@@ -55,6 +65,7 @@ struct Ctx {
 constexpr int FUSED_MAX_ROWS = 4;
 
 struct Model {
+    const ModelFamily* family;
     rotor_b200_model_config cfg;
     rotor_b200_layer_weights* layers;
     const __nv_bfloat16* embed;
@@ -97,10 +108,8 @@ struct Carve {
     }
 };
 
-// One forward over ids (device [batch * seq]) of a layer-described decoder; same contract as the ternary
-// model's run_layers: the cached lengths are read from m.c.d_pos.
-int run_decoder(Model& m, const long long* ids, int batch, int seq, int logits_mode, float* logits,
-                long long* next_ids, cudaStream_t st, bool advance);
-void destroy_decoder(DecoderStack* d);
+int launch_set_pos(int* pos, int n, int v, const int* lens, cudaStream_t st);
+// logs the picked tokens and moves every position on by one
+int launch_advance(Model& m, const long long* picked, int batch, cudaStream_t st);
 
 }  // namespace rb

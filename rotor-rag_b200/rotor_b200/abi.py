@@ -12,6 +12,9 @@ import os
 
 _HERE = os.path.dirname(os.path.abspath(__file__))
 LIB_PATH = os.path.join(_HERE, "librotor_b200.so")
+# the subset of the library that serves layer-described decoders (`make decoder`), taken where the whole
+# one has not been built
+DECODER_LIB_PATH = os.path.join(_HERE, "librotor_b200_decoder.so")
 
 OK = 0
 VARIANT_AUTO, VARIANT_DP4A, VARIANT_MMA = 0, 1, 2
@@ -25,6 +28,8 @@ class RotorB200Error(RuntimeError):
 
 def _load():
     if not os.path.exists(LIB_PATH):
+        if os.path.exists(DECODER_LIB_PATH):
+            return C.CDLL(DECODER_LIB_PATH)
         raise RotorB200Error(
             f"{LIB_PATH} not found: build it with `make -C rotor-rag_b200/csrc` "
             "(or __graft_entry__.build()); there is no CPU fallback")
@@ -149,6 +154,8 @@ _SIGNATURES.update({
 
 def _declare(signatures):
     for name, (res, args) in signatures.items():
+        if not os.path.exists(LIB_PATH) and not hasattr(lib, name):
+            continue             # the subset: calling what it leaves out raises AttributeError
         fn = getattr(lib, name)  # AttributeError here = header and library out of step
         fn.restype = res
         fn.argtypes = args
