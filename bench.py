@@ -33,6 +33,7 @@ One JSON line is printed by rank 0:
                bounded sample (N = 1 only)
 --impl reference times the reference itself on the host cores (its installed copy under baseline/_ref,
 through its own TextGenerator.generate; the port stands in where the copy is absent).
+--workload likerax times the Likerax design beside the ternary model at equal sizes.
 --workload / --only select one section alone (profiling aids; they print their own line).
 """
 import argparse
@@ -837,6 +838,193 @@ def run_xl_tp(args, rank, world):
         dist.destroy_process_group()
 
 
+def likerax_random(cfg, layers, chunk, streams=2, seed=0, **kw):
+    """A Likerax model of a BitNet shape's sizes (heads, head size, FFN, vocabulary), random weights."""
+    import torch
+    from rotor_b200.decoder_model import Connections, DecoderModel, LayerSpec
+    from rotor_b200.likerax import distance_slopes
+    g = torch.Generator(device="cuda")
+    g.manual_seed(seed)
+    d, ff, h, kv = cfg["d_model"], cfg["d_ff"], cfg["n_heads"], cfg["n_kv_heads"]
+    hd = d // h
+    mat = lambda o, i: (torch.randn((o, i), generator=g, device="cuda") / i ** 0.5).to(torch.bfloat16)
+    def hc():
+        return Connections(torch.full((streams,), 1.0 / streams), torch.ones(streams), torch.eye(streams))
+    specs = [LayerSpec(h, kv, hd, hd, hd ** -0.5, mat(h * hd, d), mat(kv * hd, d), mat(kv * hd, d), mat(d, h * hd), torch.ones(d),
+                       unit_qk=True, chunk=chunk, slopes=distance_slopes(h), gate=mat(ff, d), up=mat(ff, d), down=mat(d, ff),
+                       norm2=torch.ones(d), hc1=hc(), hc2=hc()) for _ in range(layers)]
+    return DecoderModel(specs, list(range(layers)), mat(cfg["vocab_size"], d), mat(cfg["vocab_size"], d), torch.ones(d),
+                        streams=streams, eps=1e-5, **kw)
+
+
+def time_graph(torch, run, n, iters=10):
+    """Seconds per call of `run(i)`, i = 0 .. n - 1 captured back to back in one CUDA graph."""
+    st = torch.cuda.Stream()
+    with torch.cuda.stream(st):
+        for i in range(n):
+            run(i, st.cuda_stream)
+        st.synchronize()
+        g = torch.cuda.CUDAGraph()
+        with torch.cuda.graph(g, stream=st):
+            for i in range(n):
+                run(i, st.cuda_stream)
+        for _ in range(3):
+            g.replay()
+        st.synchronize()
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        e0.record(st)
+        for _ in range(iters):
+            g.replay()
+        e1.record(st)
+        st.synchronize()
+    return e0.elapsed_time(e1) * 1e-3 / (iters * n)
+
+
+def likerax_kernels(torch, abi, cfg, B, S, chunk, streams=2):
+    """The decoder kernels alone, inputs larger than L2 (several distinct weight matrices per graph)."""
+    import ctypes as C
+    lib = abi.lib
+    with open(os.path.join(ROOT, "MEASURED_PEAKS.json")) as f:
+        peaks = json.load(f)
+    hbm, tflops = peaks["hbm_gbs"] * 1e9, peaks["bf16_tflops"] * 1e12
+    d, ff, h, kv = cfg["d_model"], cfg["d_ff"], cfg["n_heads"], cfg["n_kv_heads"]
+    hd, rows = d // h, B * S
+    qkv = (h + 2 * kv) * hd
+    bf = lambda *s: torch.randn(*s, device="cuda", dtype=torch.bfloat16)
+    out = {}
+
+    def record(name, sec, nbytes=None, flops=None):
+        r = {"us": sec * 1e6}
+        if nbytes:
+            r.update(bytes=nbytes, gbs=nbytes / sec / 1e9, frac_of_measured_hbm=nbytes / sec / hbm)
+        if flops:
+            r.update(flops=flops, tflops=flops / sec / 1e12, frac_of_measured_bf16=flops / sec / tflops)
+        out[name] = r
+
+    def product(name, n, k, gated, m):
+        nm = max(2, min(16, int(4e8 // (n * (1 + gated) * k * 2))))
+        ws = [bf(n * (1 + gated), k) / k ** 0.5 for _ in range(nm)]
+        x = bf(m, k)
+        ldn = (n + 63) // 64 * 64
+        y = torch.empty((m, ldn), device="cuda", dtype=torch.bfloat16 if gated else torch.float32)
+        sec = time_graph(torch, lambda i, s: abi.check(lib.rotor_b200_dense_linear(ws[i].data_ptr(), n, k, x.data_ptr(), m, 0, gated,
+                                                                                     y.data_ptr(), None, s)), nm)
+        if m <= 4:
+            record(name, sec, nbytes=n * (1 + gated) * k * 2)
+        else:
+            record(name, sec, flops=2.0 * m * n * (1 + gated) * k)
+
+    product("gemv_qkv", qkv, d, 0, 1)
+    product("gemv_o", d, d, 0, 1)
+    product("gemv_gate_up", ff, d, 1, 1)
+    product("gemv_down", d, ff, 0, 1)
+    product("gemm_qkv", qkv, d, 0, rows)
+    product("gemm_o", d, d, 0, rows)
+    product("gemm_gate_up", ff, d, 1, rows)
+    product("gemm_down", d, ff, 0, rows)
+    # attention: prompt (with the stand-alone head finish in front) and one token behind a long cache
+    c = abi.DecoderLayer(heads=h, kv_heads=kv, dim=hd, vdim=hd, unit_qk=1, chunk=chunk, scale=hd ** -0.5)
+    sl = torch.tensor([2.0 ** (-8 * (i + 1) / h) for i in range(h)], device="cuda")
+    c.slopes = sl.data_ptr()
+    kc, vc = bf(B, kv, S + 1, hd), bf(B, kv, S + 1, hd)
+    raw = torch.randn((rows, (qkv + 63) // 64 * 64), device="cuda")
+    o, q = bf(rows, h * hd), bf(rows, h * hd)
+    past = torch.zeros(B, dtype=torch.int32, device="cuda")
+    att = lambda seq, p: lambda i, s: abi.check(lib.rotor_b200_bias_attention(C.byref(c), 1e-5, 0, raw.data_ptr(), B, seq, p.data_ptr(), S + 1,
+                                                                                 kc.data_ptr(), vc.data_ptr(), o.data_ptr(), 0, q.data_ptr(), s))
+    seen = S * (S + 1) // 2 if chunk <= 0 or chunk >= S else \
+        S // chunk * (chunk * (chunk + 1) // 2) + (S % chunk) * (S % chunk + 1) // 2
+    record("attention_prompt_with_head_finish", time_graph(torch, att(S, past), 2), flops=4.0 * B * h * seen * hd)
+    pl = torch.full((B,), S, dtype=torch.int32, device="cuda")
+    reach = S + 1 if chunk <= 0 else S % chunk + 1
+    record("attention_token_batch", time_graph(torch, att(1, pl), 16), nbytes=2 * B * kv * reach * hd * 2)
+    # residual stage
+    x0, x1, y = (torch.randn((rows, streams, d), device="cuda"), torch.empty((rows, streams, d), device="cuda"),
+                 torch.randn((rows, d), device="cuda"))
+    mix, one = torch.eye(streams, device="cuda"), torch.ones(max(d, 64), device="cuda")
+    hh = bf(rows, d)
+    sec = time_graph(torch, lambda i, s: abi.check(lib.rotor_b200_stream_stage(
+        None, None, 0, x0.data_ptr(), x1.data_ptr(), y.data_ptr(), mix.data_ptr(), one.data_ptr(), one.data_ptr(), one.data_ptr(), 1e-5, rows,
+        streams, d, hh.data_ptr(), 0, s)), 2)
+    record("stream_stage", sec, nbytes=rows * d * (streams * 8 + 4 + 2))
+    abi.device_status()
+    return out
+
+
+def run_likerax(args):
+    """--workload likerax: prefill and decode throughput of the Likerax design beside the ternary model at
+    equal sizes (random weights; the ternary model's float work per token is the same, its weights are 2 bits)."""
+    import torch
+    from rotor_b200 import abi, semantics
+    from rotor_b200.synth import XL_TP, random_model_on_device
+    torch.cuda.set_device(0)
+    barrier = torch.cuda.synchronize
+    K, W = args.steps, max(args.warmup, 3)
+    prompt_len, S = XL_PROMPT_LEN, args.seq or 2048
+    shapes = {"2b": (dict(CFG_2B), args.layers or 6, args.batch or 8), "xl": (dict(XL_TP), min(args.layers or 2, 4), args.batch or 2)}
+    line = {"metric": "Likerax prefill and decode tokens/s beside the ternary model at equal size", "unit": UNIT, "n_gpus": 1,
+            "steps": K, "warmup": W, "higher_is_better": True, "data": "synthetic", "dtype": "bf16 (float32 residual, scores, norms)",
+            "shapes": {}}
+    before = abi.lib.rotor_b200_launch_count()
+    for name, (cfg, layers, B) in shapes.items():
+        if args.only in shapes and args.only != name:
+            continue
+        cfg["n_layers"] = layers
+        rec = {"config": dict(cfg, streams=2, chunk=args.chunk, prefill=f"{B} x {S}", decode=f"after {prompt_len} tokens")}
+        for family in ("likerax", "bitnet"):
+            if args.family not in ("both", family):
+                continue
+            max_seq = max(S, prompt_len + 1 + W + K + 8)
+            kw = dict(max_seq=max_seq, max_batch=B, max_rows=B * S)
+            model = likerax_random(cfg, layers, args.chunk, **kw) if family == "likerax" else \
+                random_model_on_device(cfg, seed=3, semantics=semantics.BASELINE, **kw)
+            r = {}
+            if args.phase in ("both", "prefill"):
+                r["prefill"] = time_prefill(torch, abi, model, cfg["vocab_size"], B, S, 5, 3)
+            if args.phase in ("both", "decode"):
+                r["decode"] = {}
+                for b in ([1, 8] if B >= 8 else [1, B]):
+                    import numpy as np
+                    h = model._ensure_handle(b, prompt_len, max_seq)
+                    ids = np.random.default_rng(7).integers(0, cfg["vocab_size"], size=(b, prompt_len)).astype(np.int64)
+                    sec, n, clocks, _ = time_decode(torch, abi, h.h, b, ids, W, K, args.graph, barrier, 0)
+                    r["decode"][str(b)] = {"tokens_per_s": b * K / sec, "us_per_step": sec * 1e6 / K, "launches_per_step": n / K,
+                                           "clocks": clocks}
+            rec[family] = r
+            del model
+            h = None
+            torch.cuda.empty_cache()
+        if args.family == "both" and args.phase == "both":
+            rec["likerax_kernels"] = likerax_kernels(torch, abi, cfg, B, S, args.chunk)
+            torch.cuda.empty_cache()
+        line["shapes"][name] = rec
+    line["gpu_launches"] = int(abi.lib.rotor_b200_launch_count() - before)
+    print(json.dumps(line), flush=True)
+
+
+def time_prefill(torch, abi, model, vocab, B, S, K, W):
+    import numpy as np
+    h = model._ensure_handle(B, S, S).h
+    ids = torch.from_numpy(np.random.default_rng(5).integers(0, vocab, size=(B, S))).cuda()
+    nxt = torch.empty(B, dtype=torch.int64, device="cuda")
+    st = torch.cuda.Stream()
+    with torch.cuda.stream(st):
+        run = lambda: abi.check(abi.lib.rotor_b200_model_forward(h, ids.data_ptr(), B, S, 0, abi.LOGITS_NONE, None, nxt.data_ptr(),
+                                                                 st.cuda_stream), "prefill")
+        for _ in range(W):
+            run()
+        st.synchronize()
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        e0.record(st)
+        for _ in range(K):
+            run()
+        e1.record(st)
+        st.synchronize()
+    abi.device_status()
+    sec = e0.elapsed_time(e1) * 1e-3 / K
+    return {"tokens_per_s": B * S / sec, "ms": sec * 1e3}
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -845,15 +1033,18 @@ def main():
     ap.add_argument("--impl", default="b200", choices=["b200", "reference"])
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--quick", action="store_true", help="headline sections only (no parity / FFN / prefill / XL records)")
-    ap.add_argument("--only", default="all", choices=["all", "decode", "gemv", "gemm"],
+    ap.add_argument("--only", default="all", choices=["all", "decode", "gemv", "gemm", "2b", "xl"],
                     help="profiling aid: run only the device-resident decode section, the GEMV section, or one "
-                         "prefill GEMM (--m tokens)")
+                         "prefill GEMM (--m tokens); --workload likerax: one shape")
     ap.add_argument("--m", type=int, default=16384, help="--only gemm: activation columns (tokens)")
-    ap.add_argument("--workload", default="decode_2b", choices=["decode_2b", "xl_tp", "prefill_2b", "ffn_block"],
+    ap.add_argument("--workload", default="decode_2b", choices=["decode_2b", "xl_tp", "prefill_2b", "ffn_block", "likerax"],
                     help="decode_2b: the headline line; xl_tp: the tensor-parallel XL shape (separate line)")
     ap.add_argument("--batch", type=int, default=0, help="prefill_2b: sequences (0 = 8); xl_tp: sequences (0 = 1)")
     ap.add_argument("--seq", type=int, default=0, help="prefill_2b: positions per sequence (0 = 2048)")
     ap.add_argument("--layers", type=int, default=0, help="xl_tp: override the layer count (0 = 80)")
+    ap.add_argument("--family", default="both", choices=["both", "likerax", "bitnet"], help="likerax: which model")
+    ap.add_argument("--phase", default="both", choices=["both", "prefill", "decode"], help="likerax: which phase")
+    ap.add_argument("--chunk", type=int, default=4096, help="likerax: chunk length of the attention mask (0 = none)")
     ap.add_argument("--graph", type=int, default=1, help="xl_tp: replay the step as a CUDA graph (1) or launch it (0)")
     args = ap.parse_args()
     rank = int(os.environ.get("RANK", 0))
@@ -878,6 +1069,9 @@ def main():
         run_reference(args, rank)
     elif args.workload == "xl_tp":
         run_xl_tp(args, rank, world)
+    elif args.workload == "likerax":
+        if rank == 0:
+            run_likerax(args)
     elif args.workload == "ffn_block":
         if rank == 0:
             run_ffn_block(args)
