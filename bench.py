@@ -937,7 +937,10 @@ def likerax_kernels(torch, abi, cfg, B, S, chunk, streams=2):
     record("attention_prompt_with_head_finish", time_graph(torch, att(S, past), 2), flops=4.0 * B * h * seen * hd)
     pl = torch.full((B,), S, dtype=torch.int32, device="cuda")
     reach = S + 1 if chunk <= 0 else S % chunk + 1
-    record("attention_token_batch", time_graph(torch, att(1, pl), 16), nbytes=2 * B * kv * reach * hd * 2)
+    for b in (1, B):
+        sec = time_graph(torch, lambda i, s: abi.check(lib.rotor_b200_bias_attention(
+            C.byref(c), 1e-5, 0, raw.data_ptr(), b, 1, pl.data_ptr(), S + 1, kc.data_ptr(), vc.data_ptr(), o.data_ptr(), 0, q.data_ptr(), s)), 16)
+        record(f"attention_token_batch_{b}", sec, nbytes=2 * b * kv * reach * hd * 2)
     # residual stage
     x0, x1, y = (torch.randn((rows, streams, d), device="cuda"), torch.empty((rows, streams, d), device="cuda"),
                  torch.randn((rows, d), device="cuda"))

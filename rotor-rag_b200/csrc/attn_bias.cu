@@ -56,6 +56,49 @@ __device__ __forceinline__ void ba_store(float* p, float v) { *p = v; }
 __device__ __forceinline__ float ba_round(float v, const __nv_bfloat16*) { return round_bf16(v); }
 __device__ __forceinline__ float ba_round(float v, const float*) { return v; }
 
+// Merges the cluster's runs, every CTA a share of the outputs.  po: this CTA's un-normalised output
+// [heads][stride], ml: maxima [heads][1], sums at ml + HB.  All threads of the CTA call.
+template <typename T>
+__device__ __forceinline__ void ba_merge(const BiasAttn& p, const float* po, int stride, const float* ml, int HB, int nh, int head0,
+                                         int row, int rank, int ns, int tid, const T*) {
+    if (ns > 1)
+        asm volatile("barrier.cluster.arrive.release.aligned;\n\tbarrier.cluster.wait.acquire.aligned;" ::: "memory");
+    else
+        __syncthreads();
+    const int vdim = p.s.vdim;
+    T* out = static_cast<T*>(p.out) + (size_t)row * p.ld_out;
+    const int total = nh * vdim;
+    for (int idx = rank * BA_THREADS + tid; idx < total; idx += ns * BA_THREADS) {
+        const int h = idx / vdim, c = idx - h * vdim;
+        float o, l;
+        if (ns == 1) {
+            o = po[h * stride + c];
+            l = ml[HB + h];
+        } else {
+            float m[BA_MAX_SPLITS], w[BA_MAX_SPLITS], v[BA_MAX_SPLITS], M = -INFINITY;
+#pragma unroll
+            for (int k = 0; k < BA_MAX_SPLITS; ++k) {  // (all remote reads in flight together)
+                m[k] = k < ns ? ba_ld_cluster(ml + h, k) : -INFINITY;
+                w[k] = k < ns ? ba_ld_cluster(ml + HB + h, k) : 0.f;
+                v[k] = k < ns ? ba_ld_cluster(po + h * stride + c, k) : 0.f;
+            }
+#pragma unroll
+            for (int k = 0; k < BA_MAX_SPLITS; ++k) M = fmaxf(M, m[k]);
+            o = 0.f;
+            l = 0.f;
+#pragma unroll
+            for (int k = 0; k < BA_MAX_SPLITS; ++k) {
+                const float e = exp2f(m[k] - M);
+                l += e * w[k];
+                o += e * v[k];
+            }
+        }
+        ba_store(out + (size_t)(head0 + h) * vdim + c, o / l);
+    }
+    if (ns > 1)  // nobody leaves while its shared memory may still be read
+        asm volatile("barrier.cluster.arrive.release.aligned;\n\tbarrier.cluster.wait.acquire.aligned;" ::: "memory");
+}
+
 template <typename T, int NI>
 __global__ void __launch_bounds__(BA_THREADS) bias_attn_rows_kernel(const __grid_constant__ BiasRowsArgs a) {
     const BiasAttn& p = a.p;
@@ -248,38 +291,234 @@ __global__ void __launch_bounds__(BA_THREADS) bias_attn_rows_kernel(const __grid
             *reinterpret_cast<float2*>(po + h * s.vd + c) = acc[i];
         }
     }
-    // ---- merge the cluster's runs: this CTA writes every ns-th output
-    if (ns > 1)
-        asm volatile("barrier.cluster.arrive.release.aligned;\n\tbarrier.cluster.wait.acquire.aligned;" ::: "memory");
-    else
-        __syncthreads();
-    T* out = static_cast<T*>(p.out) + (size_t)row * p.ld_out;
-    const int total = nh * s.vdim;
-    for (int idx = rank * BA_THREADS + tid; idx < total; idx += ns * BA_THREADS) {
-        const int h = idx / s.vdim, c = idx - h * s.vdim;
-        float o, l;
-        if (ns == 1) {
-            o = po[h * s.vd + c];
-            l = ml[HB + h];
-        } else {
-            float m[BA_MAX_SPLITS], M = -INFINITY;
-            for (int k = 0; k < BA_MAX_SPLITS; ++k) {
-                m[k] = k < ns ? ba_ld_cluster(ml + h, k) : -INFINITY;
-                M = fmaxf(M, m[k]);
-            }
-            o = 0.f;
-            l = 0.f;
-            for (int k = 0; k < BA_MAX_SPLITS; ++k)
-                if (k < ns) {
-                    const float w = exp2f(m[k] - M);
-                    l += w * ba_ld_cluster(ml + HB + h, k);
-                    o += w * ba_ld_cluster(po + h * s.vd + c, k);
-                }
+    ba_merge(p, po, s.vd, ml, HB, nh, hk * R + h0, row, rank, ns, tid, (const T*)nullptr);
+}
+
+// The same for head sizes up to 128 (64): a warp takes a strip of keys for all H query heads of its CTA
+// and needs no shared memory until the end.  W lanes hold four columns each of a key and of the queries
+// (W = 16: the two halves of the warp take alternate keys); keys come eight per half at a time, straight
+// into registers, a batch ahead of the arithmetic.  The 8 H partial dot products are summed across the W
+// lanes by a halving exchange (each step trades half of the values with the partner lane, so that every
+// lane ends with its own scores instead of all of them), the softmax runs on those, and the weights are
+// handed out again by shuffles.  Strips are folded in shared memory, CTAs of a cluster as above.
+constexpr int BS_U = 8;  // keys per half and batch
+
+__device__ __forceinline__ float4 bs_widen(const uint2 u, const __nv_bfloat16*) { return bf16x4_to_float4(u); }
+__device__ __forceinline__ float4 bs_widen(const float4 v, const float*) { return v; }
+__device__ __forceinline__ uint2 bs_narrow(const float4 v, const __nv_bfloat16*) { return float4_to_bf16x4(v); }
+__device__ __forceinline__ float4 bs_narrow(const float4 v, const float*) { return v; }
+template <typename T> struct BsVec;
+template <> struct BsVec<__nv_bfloat16> { typedef uint2 type; };
+template <> struct BsVec<float> { typedef float4 type; };
+
+template <typename T, int W, int H>
+__global__ void __launch_bounds__(BA_THREADS, sizeof(T) == 2 ? 2 : 1) bias_attn_strips_kernel(const __grid_constant__ BiasRowsArgs a) {
+    const BiasAttn& p = a.p;
+    const HeadShape& s = p.s;
+    constexpr int C = 4 * W, N = BS_U * H, VPL = N >= W ? N / W : 1, DUP = N >= W ? 1 : W / N, HALVES = 32 / W;
+    typedef typename BsVec<T>::type Vec;
+    __shared__ __align__(16) float part[BA_WARPS][H][C];
+    __shared__ float wml[2][BA_WARPS][H], ml[2 * H];
+    const int R = s.heads / s.kv_heads;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, l = lane & (W - 1), half = lane / W, base = half * W;
+    const int ns = (int)gridDim.x, rank = (int)blockIdx.x;
+    const int hk = (int)blockIdx.y / a.head_blocks, h0 = ((int)blockIdx.y - hk * a.head_blocks) * H;
+    const int nh = min(H, R - h0);
+    const int row = a.row0 + (int)blockIdx.z, b = row / p.cache.seq;
+    const int pos = min(p.cache.past_len[b] + (row - b * p.cache.seq), p.cache.max_seq - 1);
+    const int lo = p.chunk > 0 ? pos / p.chunk * p.chunk : 0;
+    const int cached = pos + (p.append ? 0 : 1) - lo;  // keys read from the cache
+    const int per = (cached + ns * BA_WARPS - 1) / (ns * BA_WARPS);
+    const int a0 = lo + (rank * BA_WARPS + warp) * per, a1 = min(a0 + per, lo + cached);
+    const size_t head_row = ((size_t)b * s.kv_heads + hk) * p.cache.max_seq;
+    T* kc = static_cast<T*>(p.cache.k) + head_row * s.kd;
+    T* vc = static_cast<T*>(p.cache.v) + head_row * s.vd;
+    const bool kon = 4 * l < s.kd, von = 4 * l < s.vd;
+
+    Vec kv[BS_U], vv[BS_U];
+    auto fetch_k = [&](int j0) {
+#pragma unroll
+        for (int u = 0; u < BS_U; ++u) {
+            const int j = j0 + u * HALVES + half;
+            kv[u] = Vec{};
+            if (j < a1 && kon) kv[u] = *reinterpret_cast<const Vec*>(kc + (size_t)j * s.kd + 4 * l);
         }
-        ba_store(out + (size_t)(hk * R + h0 + h) * s.vdim + c, o / l);
+    };
+    auto fetch_v = [&](int j0) {
+#pragma unroll
+        for (int u = 0; u < BS_U; ++u) {
+            const int j = j0 + u * HALVES + half;
+            vv[u] = Vec{};
+            if (j < a1 && von) vv[u] = *reinterpret_cast<const Vec*>(vc + (size_t)j * s.vd + 4 * l);
+        }
+    };
+    fetch_k(a0);
+    fetch_v(a0);
+    pdl_wait();
+    pdl_trigger();
+
+    // ---- this lane's four columns of every query, divided by the row's root mean square
+    const float* raw = p.qkv + (size_t)row * p.ld_qkv;
+    auto load_raw = [&](const float* v, int len) {
+        float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (4 * l < len) x.x = __ldcg(v + 4 * l);
+        if (4 * l + 1 < len) x.y = __ldcg(v + 4 * l + 1);
+        if (4 * l + 2 < len) x.z = __ldcg(v + 4 * l + 2);
+        if (4 * l + 3 < len) x.w = __ldcg(v + 4 * l + 3);
+        return x;
+    };
+    auto finish = [&](float4 x, bool norm) {
+        float inv = 1.f;
+        if (norm) {
+            float ss = x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w;
+#pragma unroll
+            for (int m = W / 2; m > 0; m >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, m);
+            inv = 1.0f / sqrtf(ss / (float)s.dim + s.eps);
+        }
+        return make_float4(ba_round(x.x * inv, kc), ba_round(x.y * inv, kc), ba_round(x.z * inv, kc), ba_round(x.w * inv, kc));
+    };
+    float4 q[H];
+#pragma unroll
+    for (int h = 0; h < H; ++h) q[h] = h < nh ? load_raw(raw + (size_t)(hk * R + h0 + h) * s.dim, s.dim) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+    for (int h = 0; h < H; ++h) q[h] = finish(q[h], s.unit);
+
+    const float scale2 = p.scale * 1.4426950408889634f;
+    const int my_h = (VPL * l / DUP) >> 3;               // the head of this lane's scores
+    const float slope2 = p.slopes && my_h < nh ? __ldg(p.slopes + hk * R + h0 + my_h) * 1.4426950408889634f : 0.f;
+    float m_run = -INFINITY, l_run = 0.f;                // of head my_h; l_run over this lane's own scores
+    float4 o[H];
+#pragma unroll
+    for (int h = 0; h < H; ++h) o[h] = make_float4(0.f, 0.f, 0.f, 0.f);
+
+    // scores of a batch (sc: partial dot products, index h * 8 + u) -> weights; then O += weights V
+    auto batch = [&](float (&sc)[N], int j0, int end) {
+#pragma unroll
+        for (int m = W / 2, cnt = N; m > 0; m >>= 1) {
+            if (cnt > 1) {
+                cnt >>= 1;
+#pragma unroll
+                for (int i = 0; i < N / 2; ++i)
+                    if (i < cnt) {
+                        const bool up = lane & m;
+                        const float send = up ? sc[i] : sc[i + cnt], keep = up ? sc[i + cnt] : sc[i];
+                        sc[i] = keep + __shfl_xor_sync(0xffffffffu, send, m);
+                    }
+            } else {
+                sc[0] += __shfl_xor_sync(0xffffffffu, sc[0], m);
+            }
+        }
+        float top = -INFINITY;
+#pragma unroll
+        for (int i = 0; i < VPL; ++i) {
+            const int u = (VPL * l / DUP + i) & 7, j = j0 + u * HALVES + half;
+            sc[i] = j < end ? sc[i] * scale2 - slope2 * (float)(pos - j) : -INFINITY;
+            top = fmaxf(top, sc[i]);
+        }
+#pragma unroll
+        for (int m = W / H / 2; m > 0; m >>= 1) top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, m));
+        if (HALVES == 2) top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, 16));
+        const float m_new = fmaxf(m_run, top), alpha = exp2f(m_run - m_new);  // (finite: a batch has a key)
+        m_run = m_new;
+        l_run *= alpha;
+#pragma unroll
+        for (int i = 0; i < VPL; ++i) {
+            sc[i] = exp2f(sc[i] - m_new);
+            l_run += sc[i];
+        }
+#pragma unroll
+        for (int h = 0; h < H; ++h) {
+            const float al = __shfl_sync(0xffffffffu, alpha, base + h * (W / H));
+            o[h] = make_float4(o[h].x * al, o[h].y * al, o[h].z * al, o[h].w * al);
+        }
+#pragma unroll
+        for (int u = 0; u < BS_U; ++u) {
+            const float4 v = bs_widen(vv[u], kc);
+#pragma unroll
+            for (int h = 0; h < H; ++h) {
+                const int idx = h * 8 + u;
+                const float w = __shfl_sync(0xffffffffu, sc[VPL > 1 ? idx % VPL : 0], base + (VPL > 1 ? idx / VPL : idx * DUP));
+                o[h].x += w * v.x;
+                o[h].y += w * v.y;
+                o[h].z += w * v.z;
+                o[h].w += w * v.w;
+            }
+        }
+    };
+    for (int j0 = a0; j0 < a1; j0 += BS_U * HALVES) {
+        float sc[N];
+#pragma unroll
+        for (int u = 0; u < BS_U; ++u) {
+            const float4 k = bs_widen(kv[u], kc);
+#pragma unroll
+            for (int h = 0; h < H; ++h) sc[h * 8 + u] = k.x * q[h].x + k.y * q[h].y + k.z * q[h].z + k.w * q[h].w;
+        }
+        fetch_k(j0 + BS_U * HALVES);
+        batch(sc, j0, a1);
+        fetch_v(j0 + BS_U * HALVES);
     }
-    if (ns > 1)  // nobody leaves while its shared memory may still be read
-        asm volatile("barrier.cluster.arrive.release.aligned;\n\tbarrier.cluster.wait.acquire.aligned;" ::: "memory");
+    if (p.append && rank == ns - 1 && warp == BA_WARPS - 1) {  // the new key and value
+        const float4 k = finish(load_raw(raw + (size_t)(s.heads + hk) * s.dim, s.dim), s.unit);
+        const float4 v = finish(load_raw(raw + (size_t)(s.heads + s.kv_heads) * s.dim + (size_t)hk * s.vdim, s.vdim), false);
+        if (h0 == 0 && half == 0) {
+            const float kf[4] = {k.x, k.y, k.z, k.w}, vf[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                if (kon) ba_store(kc + (size_t)pos * s.kd + 4 * l + e, kf[e]);
+                if (von) ba_store(vc + (size_t)pos * s.vd + 4 * l + e, vf[e]);
+            }
+        }
+        float sc[N];
+#pragma unroll
+        for (int u = 0; u < BS_U; ++u) vv[u] = u == 0 && half == 0 ? bs_narrow(v, kc) : Vec{};
+#pragma unroll
+        for (int h = 0; h < H; ++h)
+#pragma unroll
+            for (int u = 0; u < BS_U; ++u)
+                sc[h * 8 + u] = u == 0 ? k.x * q[h].x + k.y * q[h].y + k.z * q[h].z + k.w * q[h].w : 0.f;
+        batch(sc, pos, pos + 1);
+    }
+
+    // ---- fold the strips
+#pragma unroll
+    for (int m = W / H / 2; m > 0; m >>= 1) l_run += __shfl_xor_sync(0xffffffffu, l_run, m);
+    l_run *= 1.0f / DUP;
+    if (HALVES == 2) l_run += __shfl_xor_sync(0xffffffffu, l_run, 16);
+#pragma unroll
+    for (int h = 0; h < H; ++h) {
+        if (HALVES == 2) {
+            o[h].x += __shfl_xor_sync(0xffffffffu, o[h].x, 16);
+            o[h].y += __shfl_xor_sync(0xffffffffu, o[h].y, 16);
+            o[h].z += __shfl_xor_sync(0xffffffffu, o[h].z, 16);
+            o[h].w += __shfl_xor_sync(0xffffffffu, o[h].w, 16);
+        }
+        if (half == 0) *reinterpret_cast<float4*>(&part[warp][h][4 * l]) = o[h];
+    }
+    if (half == 0 && l % (W / H) == 0) {
+        wml[0][warp][my_h] = m_run;
+        wml[1][warp][my_h] = l_run;
+    }
+    __syncthreads();
+    for (int i = tid; i < H * C; i += BA_THREADS) {
+        const int h = i / C, c = i - h * C;
+        float M = -INFINITY, t = 0.f, sum = 0.f;
+#pragma unroll
+        for (int w = 0; w < BA_WARPS; ++w) M = fmaxf(M, wml[0][w][h]);
+        if (M > -INFINITY) {
+#pragma unroll
+            for (int w = 0; w < BA_WARPS; ++w) {
+                const float e = exp2f(wml[0][w][h] - M);
+                t += e * part[w][h][c];
+                sum += e * wml[1][w][h];
+            }
+        }
+        part[0][h][c] = t;  // (element read by this thread alone)
+        if (c == 0) {
+            ml[h] = M;
+            ml[H + h] = sum;
+        }
+    }
+    ba_merge(p, &part[0][0][0], C, ml, H, nh, hk * R + h0, row, rank, ns, tid, (const T*)nullptr);
 }
 
 int bias_attn_reach(const BiasAttn& p) {
@@ -293,6 +532,18 @@ static size_t ba_smem_bytes(const HeadShape& s, int hb, int tile) {
            sizeof(T) * (2 * (size_t)tile * (s.kd + pad + s.vd + pad) + s.kd + s.vd);
 }
 
+template <typename K>
+static int ba_go(K kernel, const BiasRowsArgs& a, int rows, int splits, size_t smem, cudaStream_t st) {
+    const dim3 grid(splits, a.p.s.kv_heads * a.head_blocks, rows);
+    if (a.p.append) return launch_chained(kernel, grid, dim3(BA_THREADS), smem, st, splits, a);
+    // (rows appended by the kernel just before: no early start)
+    const int pdl = g_use_pdl;
+    g_use_pdl = 0;
+    const int rc = launch_chained(kernel, grid, dim3(BA_THREADS), smem, st, splits, a);
+    g_use_pdl = pdl;
+    return rc;
+}
+
 template <typename T, int NI>
 static int ba_launch(const BiasRowsArgs& a, int rows, int splits, size_t smem, cudaStream_t st) {
     static PerDevice<bool> once;
@@ -300,14 +551,22 @@ static int ba_launch(const BiasRowsArgs& a, int rows, int splits, size_t smem, c
         RB_CUDA(cudaFuncSetAttribute(bias_attn_rows_kernel<T, NI>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)BA_SMEM_MAX));
         once.here() = true;
     }
-    const dim3 grid(splits, a.p.s.kv_heads * a.head_blocks, rows);
-    if (a.p.append) return launch_chained(bias_attn_rows_kernel<T, NI>, grid, dim3(BA_THREADS), smem, st, splits, a);
-    // (rows appended by the kernel just before: no early start)
-    const int pdl = g_use_pdl;
-    g_use_pdl = 0;
-    const int rc = launch_chained(bias_attn_rows_kernel<T, NI>, grid, dim3(BA_THREADS), smem, st, splits, a);
-    g_use_pdl = pdl;
-    return rc;
+    return ba_go(bias_attn_rows_kernel<T, NI>, a, rows, splits, smem, st);
+}
+
+template <typename T, int W>
+static int bs_launch(const BiasRowsArgs& a, int h, int rows, int splits, cudaStream_t st) {
+    switch (h) {
+        case 1: return ba_go(bias_attn_strips_kernel<T, W, 1>, a, rows, splits, 0, st);
+        case 2: return ba_go(bias_attn_strips_kernel<T, W, 2>, a, rows, splits, 0, st);
+        default: return ba_go(bias_attn_strips_kernel<T, W, 4>, a, rows, splits, 0, st);
+    }
+}
+
+static int ba_splits(long long ctas, int reach) {
+    int splits = 1;
+    while (splits < BA_MAX_SPLITS && ctas * splits <= 148 && reach >= 64 * splits) splits *= 2;
+    return splits;
 }
 
 template <typename T>
@@ -316,12 +575,20 @@ static int ba_pick(const BiasAttn& p, int row0, int rows, cudaStream_t st) {
     BiasRowsArgs a = {};
     a.p = p;
     a.row0 = row0;
-    const int R = s.heads / s.kv_heads, vp = s.vd / 2;
+    const int R = s.heads / s.kv_heads, vp = s.vd / 2, reach = bias_attn_reach(p);
+    if (s.kd <= 128 && s.vd <= 128) {
+        int h = 1;
+        while (h < R && h < 4) h *= 2;
+        a.head_block = h;
+        a.head_blocks = (R + h - 1) / h;
+        if (s.kv_heads * a.head_blocks > 65535) return ROTOR_B200_ERR_SHAPE;
+        const int splits = ba_splits((long long)rows * s.kv_heads * a.head_blocks, reach);
+        return s.kd <= 64 && s.vd <= 64 ? bs_launch<T, 16>(a, h, rows, splits, st) : bs_launch<T, 32>(a, h, rows, splits, st);
+    }
     a.head_block = R;
     const int most = BA_MAX_PAIRS * BA_THREADS / vp;
     if (most < 1) return ROTOR_B200_ERR_SHAPE;
     if (a.head_block > most) a.head_block = most;
-    const int reach = bias_attn_reach(p);
     a.tile = 128;
     for (;;) {
         while (a.tile > 32 && ba_smem_bytes<T>(s, a.head_block, a.tile) > BA_SMEM_MAX) a.tile >>= 1;
@@ -331,8 +598,7 @@ static int ba_pick(const BiasAttn& p, int row0, int rows, cudaStream_t st) {
     }
     a.head_blocks = (R + a.head_block - 1) / a.head_block;
     const long long ctas = (long long)rows * s.kv_heads * a.head_blocks;
-    int splits = 1;
-    while (splits < BA_MAX_SPLITS && ctas * splits < 296 && reach >= 64 * splits) splits *= 2;
+    const int splits = ba_splits(ctas, reach);
     // a run shorter than the tile needs no larger tile
     const int run = (reach + splits - 1) / splits;
     while (a.tile > 32 && run <= a.tile / 2) a.tile >>= 1;

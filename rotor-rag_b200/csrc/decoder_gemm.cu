@@ -22,7 +22,7 @@ namespace rb {
 template <int BN>
 struct DgT5 {
     static constexpr int A_BYTES = 128 * 128, B_BYTES = BN * 128, STAGE = A_BYTES + B_BYTES;
-    static constexpr int STAGES = BN == 256 ? 4 : 8;
+    static constexpr int STAGES = BN == 256 ? 4 : (BN == 64 ? 8 : 9);
     static constexpr int XPOSE = 4 * (int)T5_XPOSE_BYTES;
     static constexpr int SMEM = STAGES * STAGE + XPOSE + 1024;
     static constexpr int TMEM_COLS = 2 * BN;
@@ -294,7 +294,11 @@ int launch_dense_gemm_t5(const DenseProduct& p, int rows, cudaStream_t st) {
     bool wide = (long long)((rows + 127) / 128) * ((p.n + tn - 1) / tn) >= fused_sm_count();
     if (p.epilogue == DENSE_QKV && p.shape.dim > 64) wide = true;
     switch (p.epilogue) {
-        case DENSE_PLAIN: return wide ? dg5_launch<256, DENSE_PLAIN>(p, rows, st) : dg5_launch<64, DENSE_PLAIN>(p, rows, st);
+        case DENSE_PLAIN:
+            if (wide) return dg5_launch<256, DENSE_PLAIN>(p, rows, st);
+            // (a few dozen rows of a narrow output: the weight stream wants as many CTAs as there are)
+            return (long long)((rows + 127) / 128) * ((p.n + 63) / 64) * 4 >= 3LL * fused_sm_count() ? dg5_launch<64, DENSE_PLAIN>(p, rows, st)
+                                                                                                   : dg5_launch<32, DENSE_PLAIN>(p, rows, st);
         case DENSE_GATED: return wide ? dg5_launch<256, DENSE_GATED>(p, rows, st) : dg5_launch<64, DENSE_GATED>(p, rows, st);
         default: return wide ? dg5_launch<256, DENSE_QKV>(p, rows, st) : dg5_launch<64, DENSE_QKV>(p, rows, st);
     }

@@ -1,7 +1,7 @@
 // Dense products of up to four rows (generation steps): y = x W^T with bf16 weights, bound by the weight
 // stream, with the residual stage that produces x fused into the prologue and the gating into the end.
 //
-// Grid: one CTA per SM, each owning a contiguous run of output rows (a gated product: of gate / up pairs).
+// Grid: two CTAs per SM, each owning a contiguous run of output rows (a gated product: of gate / up pairs).
 // The run's work is a list of units (output row, 256 columns); the CTA's warps take equal contiguous
 // shares of that list, so that rows are split across warps where that is what balances them, and the
 // shares of a row are added in warp order (fixed order: repeated runs give identical bits).  A unit is
@@ -11,8 +11,9 @@
 
 namespace rb {
 
-constexpr int DG_THREADS = 512, DG_WARPS = DG_THREADS / 32, DG_CTAS = 148;
+constexpr int DG_THREADS = 512, DG_WARPS = DG_THREADS / 32, DG_CTAS = 296;
 constexpr int DG_U = 4;                       // units per load batch
+constexpr int DG_AHEAD = 16;                  // units requested into L2 ahead of the launch wait
 constexpr size_t DG_SMEM_MAX = 200 * 1024;
 
 struct DenseGemvArgs {
@@ -41,26 +42,38 @@ __global__ void __launch_bounds__(DG_THREADS, R <= 2 ? 2 : 1) dense_gemv_kernel(
     const int u0 = min(units, warp * upw), u1 = min(units, u0 + upw);
 
     // load cursor, a batch ahead of the arithmetic cursor
-    int lrow = u0 / steps, lstep = u0 - lrow * steps, lu = u0;
+    auto row_start = [&](int r) {
+        const int row = gated ? (r & 1) * p.n + n0 + (r >> 1) : n0 + r;
+        return p.w + (size_t)row * p.ldw + lane * 8;
+    };
+    int lrow = u0 / steps, lstep = u0 - lrow * steps, lu = u0, lcol = (lstep << 8) + lane * 8;
+    const __nv_bfloat16* lp = row_start(lrow) + (lstep << 8);
     auto fetch = [&](uint4 (&w)[DG_U]) {
 #pragma unroll
         for (int j = 0; j < DG_U; ++j) {
             w[j] = make_uint4(0u, 0u, 0u, 0u);
-            const int col = (lstep << 8) + lane * 8;
-            if (lu < u1 && col < p.ldw) {
-                const int row = gated ? (lrow & 1) * p.n + n0 + (lrow >> 1) : n0 + lrow;
-                w[j] = ld_stream_v4(reinterpret_cast<const uint4*>(p.w + (size_t)row * p.ldw + col));
-            }
+            if (lu < u1 && lcol < p.ldw) w[j] = ld_stream_v4(reinterpret_cast<const uint4*>(lp));
             ++lu;
+            lp += 256;
+            lcol += 256;
             if (++lstep == steps) {
                 lstep = 0;
-                ++lrow;
+                lcol = lane * 8;
+                lp = row_start(++lrow);
             }
         }
     };
     uint4 wa[DG_U], wb[DG_U];
     fetch(wa);
-    fetch(wb);
+    // the stream goes on during the prologue: the next units, a 128-byte line per lane, into L2
+#pragma unroll
+    for (int i = 0; i < DG_AHEAD / 8; ++i) {
+        const int u = u0 + DG_U + 8 * i + (lane >> 2);
+        if (u < u1) {
+            const int r = u / steps, col = ((u - r * steps) << 8) + (lane & 3) * 64;
+            if (col < p.ldw) prefetch_l2(row_start(r) - lane * 8 + col);
+        }
+    }
     if (a.has_stage) stream_coefs(a.st, coef);
     pdl_wait();
     pdl_trigger();
@@ -112,37 +125,54 @@ __global__ void __launch_bounds__(DG_THREADS, R <= 2 ? 2 : 1) dense_gemv_kernel(
     }
     __syncthreads();
 
-    float acc[R];
+    float acc[R], acc2[R];
 #pragma unroll
-    for (int r = 0; r < R; ++r) acc[r] = 0.f;
+    for (int r = 0; r < R; ++r) acc[r] = acc2[r] = 0.f;
     int crow = u0 / steps, cstep = u0 - crow * steps, cu = u0;
     auto flush = [&]() {
         const int slot = warp - (crow * steps) / upw;
 #pragma unroll
         for (int r = 0; r < R; ++r) {
-            const float t = warp_sum(acc[r]);
+            const float t = warp_sum(acc[r] + acc2[r]);
             if (lane == 0) part[((size_t)crow * a.slots + slot) * R + r] = t;
-            acc[r] = 0.f;
+            acc[r] = acc2[r] = 0.f;
+        }
+    };
+    auto mac = [&](const uint4& w, const float* x) {
+        const float4 wlo = bf16x4_to_float4(make_uint2(w.x, w.y)), whi = bf16x4_to_float4(make_uint2(w.z, w.w));
+#pragma unroll
+        for (int r = 0; r < R; ++r) {
+            const float4 xa = *reinterpret_cast<const float4*>(x + r * kx), xb = *reinterpret_cast<const float4*>(x + r * kx + 128);
+            acc[r] += wlo.x * xa.x;
+            acc2[r] += whi.x * xb.x;
+            acc[r] += wlo.y * xa.y;
+            acc2[r] += whi.y * xb.y;
+            acc[r] += wlo.z * xa.z;
+            acc2[r] += whi.z * xb.z;
+            acc[r] += wlo.w * xa.w;
+            acc2[r] += whi.w * xb.w;
         }
     };
     auto consume = [&](const uint4 (&w)[DG_U]) {
+        const float* x = xs + (cstep << 8) + lane * 4;
+        if (cu + DG_U <= u1 && cstep + DG_U <= steps) {  // one row, the whole batch (warp-uniform)
+#pragma unroll
+            for (int j = 0; j < DG_U; ++j) mac(w[j], x + (j << 8));
+            cu += DG_U;
+            cstep += DG_U;
+            if (cstep == steps) {
+                flush();
+                cstep = 0;
+                ++crow;
+            } else if (cu == u1) {
+                flush();
+            }
+            return;
+        }
 #pragma unroll
         for (int j = 0; j < DG_U; ++j) {
-            if (cu < u1) {  // warp-uniform
-                const float4 wlo = bf16x4_to_float4(make_uint2(w[j].x, w[j].y)), whi = bf16x4_to_float4(make_uint2(w[j].z, w[j].w));
-#pragma unroll
-                for (int r = 0; r < R; ++r) {
-                    const float* xr = xs + r * kx + (cstep << 8) + lane * 4;
-                    const float4 xa = *reinterpret_cast<const float4*>(xr), xb = *reinterpret_cast<const float4*>(xr + 128);
-                    acc[r] += wlo.x * xa.x;
-                    acc[r] += wlo.y * xa.y;
-                    acc[r] += wlo.z * xa.z;
-                    acc[r] += wlo.w * xa.w;
-                    acc[r] += whi.x * xb.x;
-                    acc[r] += whi.y * xb.y;
-                    acc[r] += whi.z * xb.z;
-                    acc[r] += whi.w * xb.w;
-                }
+            if (cu < u1) {
+                mac(w[j], xs + (cstep << 8) + lane * 4);
                 ++cu;
                 if (++cstep == steps) {
                     flush();
@@ -154,6 +184,7 @@ __global__ void __launch_bounds__(DG_THREADS, R <= 2 ? 2 : 1) dense_gemv_kernel(
             }
         }
     };
+    fetch(wb);
     while (cu < u1) {
         consume(wa);
         fetch(wa);
