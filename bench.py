@@ -859,6 +859,7 @@ def likerax_random(cfg, layers, chunk, streams=2, seed=0, **kw):
 
 def time_graph(torch, run, n, iters=10):
     """Seconds per call of `run(i)`, i = 0 .. n - 1 captured back to back in one CUDA graph."""
+    torch.cuda.synchronize()      # the inputs were made on another stream
     st = torch.cuda.Stream()
     with torch.cuda.stream(st):
         for i in range(n):
@@ -1010,6 +1011,7 @@ def time_prefill(torch, abi, model, vocab, B, S, K, W):
     h = model._ensure_handle(B, S, S).h
     ids = torch.from_numpy(np.random.default_rng(5).integers(0, vocab, size=(B, S))).cuda()
     nxt = torch.empty(B, dtype=torch.int64, device="cuda")
+    torch.cuda.synchronize()
     st = torch.cuda.Stream()
     with torch.cuda.stream(st):
         run = lambda: abi.check(abi.lib.rotor_b200_model_forward(h, ids.data_ptr(), B, S, 0, abi.LOGITS_NONE, None, nxt.data_ptr(),

@@ -60,7 +60,7 @@ __device__ __forceinline__ float ba_round(float v, const float*) { return v; }
 // [heads][stride], ml: maxima [heads][1], sums at ml + HB.  All threads of the CTA call.
 template <typename T>
 __device__ __forceinline__ void ba_merge(const BiasAttn& p, const float* po, int stride, const float* ml, int HB, int nh, int head0,
-                                         int row, int rank, int ns, int tid, const T*) {
+                                         int row, int rank, int ns, int tid, int nthr, const T*) {
     if (ns > 1)
         asm volatile("barrier.cluster.arrive.release.aligned;\n\tbarrier.cluster.wait.acquire.aligned;" ::: "memory");
     else
@@ -68,7 +68,7 @@ __device__ __forceinline__ void ba_merge(const BiasAttn& p, const float* po, int
     const int vdim = p.s.vdim;
     T* out = static_cast<T*>(p.out) + (size_t)row * p.ld_out;
     const int total = nh * vdim;
-    for (int idx = rank * BA_THREADS + tid; idx < total; idx += ns * BA_THREADS) {
+    for (int idx = rank * nthr + tid; idx < total; idx += ns * nthr) {
         const int h = idx / vdim, c = idx - h * vdim;
         float o, l;
         if (ns == 1) {
@@ -120,7 +120,7 @@ __global__ void __launch_bounds__(BA_THREADS) bias_attn_rows_kernel(const __grid
     const int hk = (int)blockIdx.y / a.head_blocks, h0 = ((int)blockIdx.y - hk * a.head_blocks) * HB;
     const int nh = min(HB, R - h0);                         // query heads of this CTA: hk R + h0 ..
     const int row = a.row0 + (int)blockIdx.z, b = row / p.cache.seq;
-    const int pos = min(p.cache.past_len[b] + (row - b * p.cache.seq), p.cache.max_seq - 1);
+    const int pos = min(cached_len(p.cache.past_len, b, p.cache.max_seq) + (row - b * p.cache.seq), p.cache.max_seq - 1);
     const int lo = p.chunk > 0 ? pos / p.chunk * p.chunk : 0;
     const int per = (pos + 1 - lo + ns - 1) / ns;
     const int t0 = lo + rank * per, t1 = min(t0 + per, pos + 1);
@@ -291,7 +291,7 @@ __global__ void __launch_bounds__(BA_THREADS) bias_attn_rows_kernel(const __grid
             *reinterpret_cast<float2*>(po + h * s.vd + c) = acc[i];
         }
     }
-    ba_merge(p, po, s.vd, ml, HB, nh, hk * R + h0, row, rank, ns, tid, (const T*)nullptr);
+    ba_merge(p, po, s.vd, ml, HB, nh, hk * R + h0, row, rank, ns, tid, BA_THREADS, (const T*)nullptr);
 }
 
 // The same for head sizes up to 128 (64): a warp takes a strip of keys for all H query heads of its CTA
@@ -311,25 +311,26 @@ template <typename T> struct BsVec;
 template <> struct BsVec<__nv_bfloat16> { typedef uint2 type; };
 template <> struct BsVec<float> { typedef float4 type; };
 
-template <typename T, int W, int H>
-__global__ void __launch_bounds__(BA_THREADS, sizeof(T) == 2 ? 2 : 1) bias_attn_strips_kernel(const __grid_constant__ BiasRowsArgs a) {
+template <typename T, int W, int H, int NW>
+__global__ void __launch_bounds__(32 * NW, sizeof(T) == 2 ? 16 / NW : 1) bias_attn_strips_kernel(const __grid_constant__ BiasRowsArgs a) {
     const BiasAttn& p = a.p;
     const HeadShape& s = p.s;
     constexpr int C = 4 * W, N = BS_U * H, VPL = N >= W ? N / W : 1, DUP = N >= W ? 1 : W / N, HALVES = 32 / W;
     typedef typename BsVec<T>::type Vec;
-    __shared__ __align__(16) float part[BA_WARPS][H][C];
-    __shared__ float wml[2][BA_WARPS][H], ml[2 * H];
+    __shared__ __align__(16) float part[NW][H][C];
+    __shared__ float wml[2][NW][H], ml[2 * H];
     const int R = s.heads / s.kv_heads;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, l = lane & (W - 1), half = lane / W, base = half * W;
     const int ns = (int)gridDim.x, rank = (int)blockIdx.x;
     const int hk = (int)blockIdx.y / a.head_blocks, h0 = ((int)blockIdx.y - hk * a.head_blocks) * H;
     const int nh = min(H, R - h0);
     const int row = a.row0 + (int)blockIdx.z, b = row / p.cache.seq;
-    const int pos = min(p.cache.past_len[b] + (row - b * p.cache.seq), p.cache.max_seq - 1);
+    const int pos = min(cached_len(p.cache.past_len, b, p.cache.max_seq) + (row - b * p.cache.seq), p.cache.max_seq - 1);
     const int lo = p.chunk > 0 ? pos / p.chunk * p.chunk : 0;
     const int cached = pos + (p.append ? 0 : 1) - lo;  // keys read from the cache
-    const int per = (cached + ns * BA_WARPS - 1) / (ns * BA_WARPS);
-    const int a0 = lo + (rank * BA_WARPS + warp) * per, a1 = min(a0 + per, lo + cached);
+    // the very last warp takes the new key, the others share the cached ones
+    const int strips = ns * NW - (p.append ? 1 : 0), per = (cached + strips - 1) / strips;
+    const int a0 = lo + (rank * NW + warp) * per, a1 = min(a0 + per, lo + cached);  // (empty for the last warp)
     const size_t head_row = ((size_t)b * s.kv_heads + hk) * p.cache.max_seq;
     T* kc = static_cast<T*>(p.cache.k) + head_row * s.kd;
     T* vc = static_cast<T*>(p.cache.v) + head_row * s.vd;
@@ -359,8 +360,13 @@ __global__ void __launch_bounds__(BA_THREADS, sizeof(T) == 2 ? 2 : 1) bias_attn_
 
     // ---- this lane's four columns of every query, divided by the row's root mean square
     const float* raw = p.qkv + (size_t)row * p.ld_qkv;
+    const bool vec = ((s.dim | s.vdim | p.ld_qkv) & 3) == 0;
     auto load_raw = [&](const float* v, int len) {
         float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (vec) {  // rows start on 16 bytes
+            if (4 * l < len) x = __ldcg(reinterpret_cast<const float4*>(v + 4 * l));
+            return x;
+        }
         if (4 * l < len) x.x = __ldcg(v + 4 * l);
         if (4 * l + 1 < len) x.y = __ldcg(v + 4 * l + 1);
         if (4 * l + 2 < len) x.z = __ldcg(v + 4 * l + 2);
@@ -457,7 +463,7 @@ __global__ void __launch_bounds__(BA_THREADS, sizeof(T) == 2 ? 2 : 1) bias_attn_
         batch(sc, j0, a1);
         fetch_v(j0 + BS_U * HALVES);
     }
-    if (p.append && rank == ns - 1 && warp == BA_WARPS - 1) {  // the new key and value
+    if (p.append && rank == ns - 1 && warp == NW - 1) {  // the new key and value
         const float4 k = finish(load_raw(raw + (size_t)(s.heads + hk) * s.dim, s.dim), s.unit);
         const float4 v = finish(load_raw(raw + (size_t)(s.heads + s.kv_heads) * s.dim + (size_t)hk * s.vdim, s.vdim), false);
         if (h0 == 0 && half == 0) {
@@ -499,14 +505,14 @@ __global__ void __launch_bounds__(BA_THREADS, sizeof(T) == 2 ? 2 : 1) bias_attn_
         wml[1][warp][my_h] = l_run;
     }
     __syncthreads();
-    for (int i = tid; i < H * C; i += BA_THREADS) {
+    for (int i = tid; i < H * C; i += 32 * NW) {
         const int h = i / C, c = i - h * C;
         float M = -INFINITY, t = 0.f, sum = 0.f;
 #pragma unroll
-        for (int w = 0; w < BA_WARPS; ++w) M = fmaxf(M, wml[0][w][h]);
+        for (int w = 0; w < NW; ++w) M = fmaxf(M, wml[0][w][h]);
         if (M > -INFINITY) {
 #pragma unroll
-            for (int w = 0; w < BA_WARPS; ++w) {
+            for (int w = 0; w < NW; ++w) {
                 const float e = exp2f(wml[0][w][h] - M);
                 t += e * part[w][h][c];
                 sum += e * wml[1][w][h];
@@ -518,7 +524,7 @@ __global__ void __launch_bounds__(BA_THREADS, sizeof(T) == 2 ? 2 : 1) bias_attn_
             ml[H + h] = sum;
         }
     }
-    ba_merge(p, &part[0][0][0], C, ml, H, nh, hk * R + h0, row, rank, ns, tid, (const T*)nullptr);
+    ba_merge(p, &part[0][0][0], C, ml, H, nh, hk * R + h0, row, rank, ns, tid, 32 * NW, (const T*)nullptr);
 }
 
 int bias_attn_reach(const BiasAttn& p) {
@@ -533,13 +539,13 @@ static size_t ba_smem_bytes(const HeadShape& s, int hb, int tile) {
 }
 
 template <typename K>
-static int ba_go(K kernel, const BiasRowsArgs& a, int rows, int splits, size_t smem, cudaStream_t st) {
+static int ba_go(K kernel, const BiasRowsArgs& a, int rows, int splits, size_t smem, cudaStream_t st, int threads = BA_THREADS) {
     const dim3 grid(splits, a.p.s.kv_heads * a.head_blocks, rows);
-    if (a.p.append) return launch_chained(kernel, grid, dim3(BA_THREADS), smem, st, splits, a);
+    if (a.p.append) return launch_chained(kernel, grid, dim3(threads), smem, st, splits, a);
     // (rows appended by the kernel just before: no early start)
     const int pdl = g_use_pdl;
     g_use_pdl = 0;
-    const int rc = launch_chained(kernel, grid, dim3(BA_THREADS), smem, st, splits, a);
+    const int rc = launch_chained(kernel, grid, dim3(threads), smem, st, splits, a);
     g_use_pdl = pdl;
     return rc;
 }
@@ -554,18 +560,27 @@ static int ba_launch(const BiasRowsArgs& a, int rows, int splits, size_t smem, c
     return ba_go(bias_attn_rows_kernel<T, NI>, a, rows, splits, smem, st);
 }
 
-template <typename T, int W>
+template <typename T, int W, int NW>
 static int bs_launch(const BiasRowsArgs& a, int h, int rows, int splits, cudaStream_t st) {
     switch (h) {
-        case 1: return ba_go(bias_attn_strips_kernel<T, W, 1>, a, rows, splits, 0, st);
-        case 2: return ba_go(bias_attn_strips_kernel<T, W, 2>, a, rows, splits, 0, st);
-        default: return ba_go(bias_attn_strips_kernel<T, W, 4>, a, rows, splits, 0, st);
+        case 1: return ba_go(bias_attn_strips_kernel<T, W, 1, NW>, a, rows, splits, 0, st, 32 * NW);
+        case 2: return ba_go(bias_attn_strips_kernel<T, W, 2, NW>, a, rows, splits, 0, st, 32 * NW);
+        default: return ba_go(bias_attn_strips_kernel<T, W, 4, NW>, a, rows, splits, 0, st, 32 * NW);
     }
+}
+template <typename T, int W>
+static int bs_pick(const BiasRowsArgs& a, int h, int rows, int splits, int reach, cudaStream_t st) {
+    // few CTAs and long runs: twice the warps per CTA
+    if constexpr (sizeof(T) == 2)
+        if ((long long)rows * a.p.s.kv_heads * a.head_blocks * splits <= 148 && reach >= 128 * splits)
+            return bs_launch<T, W, 16>(a, h, rows, splits, st);
+    return bs_launch<T, W, 8>(a, h, rows, splits, st);
 }
 
 static int ba_splits(long long ctas, int reach) {
+    // (clusters of eight do not fill every GPC: beyond about a hundred CTAs some would wait for a second round)
     int splits = 1;
-    while (splits < BA_MAX_SPLITS && ctas * splits <= 148 && reach >= 64 * splits) splits *= 2;
+    while (splits < BA_MAX_SPLITS && ctas * splits * 2 <= (splits == 4 ? 96 : 148) && reach >= 64 * splits) splits *= 2;
     return splits;
 }
 
@@ -583,7 +598,7 @@ static int ba_pick(const BiasAttn& p, int row0, int rows, cudaStream_t st) {
         a.head_blocks = (R + h - 1) / h;
         if (s.kv_heads * a.head_blocks > 65535) return ROTOR_B200_ERR_SHAPE;
         const int splits = ba_splits((long long)rows * s.kv_heads * a.head_blocks, reach);
-        return s.kd <= 64 && s.vd <= 64 ? bs_launch<T, 16>(a, h, rows, splits, st) : bs_launch<T, 32>(a, h, rows, splits, st);
+        return s.kd <= 64 && s.vd <= 64 ? bs_pick<T, 16>(a, h, rows, splits, reach, st) : bs_pick<T, 32>(a, h, rows, splits, reach, st);
     }
     a.head_block = R;
     const int most = BA_MAX_PAIRS * BA_THREADS / vp;

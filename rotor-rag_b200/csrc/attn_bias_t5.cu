@@ -61,7 +61,7 @@ attn_bias_t5_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_const
     const int G = p.heads / p.kv_heads, QT = B5_BM / G;
     const int qt = gridDim.x - 1 - blockIdx.x;  // late query tiles tend to see more keys: start them first
     const int hk = blockIdx.y, b = blockIdx.z, s0 = qt * QT;
-    const int past = p.past_len[b];
+    const int past = cached_len(p.past_len, b, p.max_seq);
     volatile int* abort_flag = &s_abort;
     const int s_last = min(s0 + QT, p.seq) - 1;
     const int p0 = past + s0;

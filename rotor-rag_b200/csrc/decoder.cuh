@@ -149,6 +149,10 @@ inline int launch_chained(void (*kernel)(KArgs...), dim3 grid, dim3 block, size_
 }
 
 #ifdef __CUDACC__
+// Cached length of sequence b, kept inside the cache whatever the word holds.
+__device__ __forceinline__ int cached_len(const int* past_len, int b, int max_seq) {
+    return min(max(__ldg(past_len + b), 0), max_seq - 1);
+}
 __device__ __forceinline__ float round_bf16(float v) { return __bfloat162float(__float2bfloat16_rn(v)); }
 __device__ __forceinline__ float4 bf16x4_to_float4(const uint2 u) {
     return make_float4(__uint_as_float(u.x << 16), __uint_as_float(u.x & 0xffff0000u), __uint_as_float(u.y << 16),
@@ -164,65 +168,52 @@ __device__ __forceinline__ float gelu_tanh(float z) {
     return z / (1.0f + expf(fminf(t, 80.f)));
 }
 
-// Four columns (group g) of a stage's new streams; returns their part of u.  `coef` (shared memory):
-// mix [streams][streams], out [streams], in [streams].  S = 0: any number of streams.
+// Four columns (group g) of a stage's row, in two steps so that a thread can request several groups before
+// it uses the first: the loads, then the new streams and their part of u.  `coef` (shared memory):
+// mix [streams][streams], out [streams], in [streams].  S = 0: any number of streams (old streams are loaded
+// in the second step).
 template <int S>
-__device__ __forceinline__ float4 stream_group(const StreamStage& p, const float* coef, int row, int g, bool write) {
-    const int ns = S ? S : p.streams;
-    const float* mix = coef;
-    const float* out = coef + ns * ns;
-    const float* in = out + ns;
-    float4 u = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (p.ids) {
-        long long id = p.ids[row];
-        if (id < 0 || id >= p.vocab) id = 0;
-        const float4 e = bf16x4_to_float4(__ldg(reinterpret_cast<const uint2*>(p.embed + (size_t)id * p.ld) + g));
-#pragma unroll
-        for (int t = 0; t < ns; ++t) {
-            u.x += in[t] * e.x;
-            u.y += in[t] * e.y;
-            u.z += in[t] * e.z;
-            u.w += in[t] * e.w;
-            if (write) reinterpret_cast<float4*>(p.x_out + ((size_t)row * ns + t) * p.ld)[g] = e;
+struct StreamGroup {
+    float4 y, x[S ? S : 1];  // (a first stage keeps the embedding's columns in y)
+    __device__ __forceinline__ void load(const StreamStage& p, int row, int g) {
+        if (p.ids) {
+            long long id = p.ids[row];
+            if (id < 0 || id >= p.vocab) id = 0;
+            y = bf16x4_to_float4(__ldg(reinterpret_cast<const uint2*>(p.embed + (size_t)id * p.ld) + g));
+            return;
         }
-        return u;
+        y = __ldcg(reinterpret_cast<const float4*>(p.y + (size_t)row * p.ld) + g);
+        if constexpr (S > 0) {
+            const float* xr = p.x_in + (size_t)row * S * p.ld;
+#pragma unroll
+            for (int s = 0; s < S; ++s) x[s] = __ldcg(reinterpret_cast<const float4*>(xr + (size_t)s * p.ld) + g);
+        }
     }
-    const float4 y = __ldcg(reinterpret_cast<const float4*>(p.y + (size_t)row * p.ld) + g);
-    const float* xr = p.x_in + (size_t)row * ns * p.ld;
-    if constexpr (S > 0) {
-        float4 x[S];
+    __device__ __forceinline__ float4 finish(const StreamStage& p, const float* coef, int row, int g, bool write) const {
+        const int ns = S ? S : p.streams;
+        const float* mix = coef;
+        const float* out = coef + ns * ns;
+        const float* in = out + ns;
+        float4 u = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
-        for (int s = 0; s < S; ++s) x[s] = __ldcg(reinterpret_cast<const float4*>(xr + (size_t)s * p.ld) + g);
-#pragma unroll
-        for (int t = 0; t < S; ++t) {
-            const float o = out[t];
-            float4 v = make_float4(o * y.x, o * y.y, o * y.z, o * y.w);
-#pragma unroll
-            for (int s = 0; s < S; ++s) {
-                const float m = mix[s * S + t];
-                v.x += m * x[s].x;
-                v.y += m * x[s].y;
-                v.z += m * x[s].z;
-                v.w += m * x[s].w;
-            }
-            if (write) reinterpret_cast<float4*>(p.x_out + ((size_t)row * S + t) * p.ld)[g] = v;
-            const float i = in[t];
-            u.x += i * v.x;
-            u.y += i * v.y;
-            u.z += i * v.z;
-            u.w += i * v.w;
-        }
-    } else {
         for (int t = 0; t < ns; ++t) {
-            const float o = out[t];
-            float4 v = make_float4(o * y.x, o * y.y, o * y.z, o * y.w);
-            for (int s = 0; s < ns; ++s) {
-                const float m = mix[s * ns + t];
-                const float4 x = __ldcg(reinterpret_cast<const float4*>(xr + (size_t)s * p.ld) + g);
-                v.x += m * x.x;
-                v.y += m * x.y;
-                v.z += m * x.z;
-                v.w += m * x.w;
+            float4 v = y;
+            if (!p.ids) {
+                const float o = out[t];
+                v = make_float4(o * y.x, o * y.y, o * y.z, o * y.w);
+#pragma unroll
+                for (int s = 0; s < ns; ++s) {
+                    const float m = mix[s * ns + t];
+                    float4 xs;
+                    if constexpr (S > 0)
+                        xs = x[s];
+                    else
+                        xs = __ldcg(reinterpret_cast<const float4*>(p.x_in + ((size_t)row * ns + s) * p.ld) + g);
+                    v.x += m * xs.x;
+                    v.y += m * xs.y;
+                    v.z += m * xs.z;
+                    v.w += m * xs.w;
+                }
             }
             if (write) reinterpret_cast<float4*>(p.x_out + ((size_t)row * ns + t) * p.ld)[g] = v;
             const float i = in[t];
@@ -231,9 +222,9 @@ __device__ __forceinline__ float4 stream_group(const StreamStage& p, const float
             u.z += i * v.z;
             u.w += i * v.w;
         }
+        return u;
     }
-    return u;
-}
+};
 
 // The stage's coefficients into shared memory (they are weights: may run before the launch wait).
 __device__ __forceinline__ void stream_coefs(const StreamStage& p, float* coef) {

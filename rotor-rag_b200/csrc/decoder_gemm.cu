@@ -219,7 +219,7 @@ dense_gemm_t5_kernel(const __grid_constant__ CUtensorMap tm_a, const __grid_cons
                         const int tok = tok0 + tl;
                         if (tok >= p.rows) return nullptr;
                         if (kind == 0) return p.q + (size_t)tok * dq + col;  // (kd == dim)
-                        const int b = tok / p.cache.seq, pos = __ldg(p.cache.past_len + b) + (tok - b * p.cache.seq);
+                        const int b = tok / p.cache.seq, pos = cached_len(p.cache.past_len, b, p.cache.max_seq) + (tok - b * p.cache.seq);
                         if (pos >= p.cache.max_seq) return nullptr;
                         __nv_bfloat16* base = static_cast<__nv_bfloat16*>(kind == 1 ? p.cache.k : p.cache.v);
                         return base + (((size_t)b * p.s.kv_heads + head) * p.cache.max_seq + pos) * wide + off;

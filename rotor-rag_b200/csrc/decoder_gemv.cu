@@ -74,7 +74,16 @@ __global__ void __launch_bounds__(DG_THREADS, R <= 2 ? 2 : 1) dense_gemv_kernel(
             if (col < p.ldw) prefetch_l2(row_start(r) - lane * 8 + col);
         }
     }
-    if (a.has_stage) stream_coefs(a.st, coef);
+    constexpr int SG = 2;  // column groups per thread requested together
+    float4 nw[SG];
+    if (a.has_stage) {
+        stream_coefs(a.st, coef);
+#pragma unroll
+        for (int i = 0; i < SG; ++i) {
+            const int g = threadIdx.x + i * DG_THREADS;
+            nw[i] = g < (a.st.ld >> 2) ? __ldg(reinterpret_cast<const float4*>(a.st.norm) + g) : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+    }
     pdl_wait();
     pdl_trigger();
     __syncthreads();
@@ -85,42 +94,61 @@ __global__ void __launch_bounds__(DG_THREADS, R <= 2 ? 2 : 1) dense_gemv_kernel(
         int k = 0;
         for (int r = 0; r < R; ++r) {
             float ss = 0.f;
-            for (int g = threadIdx.x; g < (kx >> 2); g += DG_THREADS) {
-                float4 u = make_float4(0.f, 0.f, 0.f, 0.f);
-                if (g < n4) {
-                    u = stream_group<S>(s, coef, r, g, g % gridDim.x == blockIdx.x);
-                    ss += u.x * u.x + u.y * u.y + u.z * u.z + u.w * u.w;
+            for (int g0 = threadIdx.x; g0 < (kx >> 2); g0 += SG * DG_THREADS) {
+                StreamGroup<S> sg[SG];
+#pragma unroll
+                for (int i = 0; i < SG; ++i)
+                    if (g0 + i * DG_THREADS < n4) sg[i].load(s, r, g0 + i * DG_THREADS);
+#pragma unroll
+                for (int i = 0; i < SG; ++i) {
+                    const int g = g0 + i * DG_THREADS;
+                    float4 u = make_float4(0.f, 0.f, 0.f, 0.f);
+                    if (g < n4) {
+                        u = sg[i].finish(s, coef, r, g, g % gridDim.x == blockIdx.x);
+                        ss += u.x * u.x + u.y * u.y + u.z * u.z + u.w * u.w;
+                    }
+                    if (g < (kx >> 2)) *reinterpret_cast<float4*>(xs + r * kx + dg_slot(g << 2)) = u;
                 }
-                *reinterpret_cast<float4*>(xs + r * kx + dg_slot(g << 2)) = u;
             }
             ss = block_sum_alt(ss, red, k);
             const float inv = 1.0f / sqrtf(ss / (float)s.n + s.eps);
-            for (int g = threadIdx.x; g < n4; g += DG_THREADS) {  // own groups
+            auto scale = [&](int g, const float4 w) {  // own groups
                 float4* q = reinterpret_cast<float4*>(xs + r * kx + dg_slot(g << 2));
-                const float4 w = __ldg(reinterpret_cast<const float4*>(s.norm) + g);
                 float4 v = *q;
                 v = make_float4(v.x * inv * w.x, v.y * inv * w.y, v.z * inv * w.z, v.w * inv * w.w);
                 if (!p.f32) v = make_float4(round_bf16(v.x), round_bf16(v.y), round_bf16(v.z), round_bf16(v.w));
                 *q = v;
-            }
+            };
+#pragma unroll
+            for (int i = 0; i < SG; ++i)
+                if ((int)threadIdx.x + i * DG_THREADS < n4) scale(threadIdx.x + i * DG_THREADS, nw[i]);
+            for (int g = threadIdx.x + SG * DG_THREADS; g < n4; g += DG_THREADS)
+                scale(g, __ldg(reinterpret_cast<const float4*>(s.norm) + g));
         }
     } else {
+        constexpr int XG = 4;
         for (int r = 0; r < R; ++r)
-            for (int g = threadIdx.x; g < (kx >> 2); g += DG_THREADS) {
-                float v[4] = {0.f, 0.f, 0.f, 0.f};
-                const int c = g << 2;
-                if (c < p.k) {
-                    float4 f;
+            for (int g0 = threadIdx.x; g0 < (kx >> 2); g0 += XG * DG_THREADS) {
+                float4 f[XG];
+#pragma unroll
+                for (int i = 0; i < XG; ++i) {
+                    const int g = g0 + i * DG_THREADS;
+                    f[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+                    if ((g << 2) >= p.k) continue;
                     if (p.f32)
-                        f = __ldcg(reinterpret_cast<const float4*>(static_cast<const float*>(p.x) + (size_t)r * p.ldx) + g);
+                        f[i] = __ldcg(reinterpret_cast<const float4*>(static_cast<const float*>(p.x) + (size_t)r * p.ldx) + g);
                     else
-                        f = bf16x4_to_float4(__ldcg(reinterpret_cast<const uint2*>(static_cast<const __nv_bfloat16*>(p.x) + (size_t)r * p.ldx) + g));
-                    v[0] = f.x;
-                    v[1] = c + 1 < p.k ? f.y : 0.f;  // (pad columns of the row may hold another product's values)
-                    v[2] = c + 2 < p.k ? f.z : 0.f;
-                    v[3] = c + 3 < p.k ? f.w : 0.f;
+                        f[i] = bf16x4_to_float4(__ldcg(reinterpret_cast<const uint2*>(static_cast<const __nv_bfloat16*>(p.x) + (size_t)r * p.ldx) + g));
                 }
-                *reinterpret_cast<float4*>(xs + r * kx + dg_slot(c)) = make_float4(v[0], v[1], v[2], v[3]);
+#pragma unroll
+                for (int i = 0; i < XG; ++i) {
+                    const int c = (g0 + i * DG_THREADS) << 2;
+                    if (c >= kx) continue;
+                    if (c + 1 >= p.k) f[i].y = 0.f;  // (pad columns of the row may hold another product's values)
+                    if (c + 2 >= p.k) f[i].z = 0.f;
+                    if (c + 3 >= p.k) f[i].w = 0.f;
+                    *reinterpret_cast<float4*>(xs + r * kx + dg_slot(c)) = f[i];
+                }
             }
     }
     __syncthreads();

@@ -20,7 +20,9 @@ __global__ void __launch_bounds__(256) stream_stage_kernel(const __grid_constant
         const int src = p.row_map ? p.row_map[r] : r;
         float ss = 0.f;
         for (int g = threadIdx.x; g < n4; g += blockDim.x) {
-            const float4 u = stream_group<S>(p, coef, src, g, p.x_out != nullptr);
+            StreamGroup<S> sg;
+            sg.load(p, src, g);
+            const float4 u = sg.finish(p, coef, src, g, p.x_out != nullptr);
             ss += u.x * u.x + u.y * u.y + u.z * u.z + u.w * u.w;
             reinterpret_cast<float4*>(us)[g] = u;
         }
@@ -82,7 +84,7 @@ __global__ void __launch_bounds__(256) head_finish_kernel(const __grid_constant_
         if (v < s.heads) {
             dst = ((size_t)row * s.heads + v) * s.kd;
         } else {
-            const int b = row / p.cache.seq, pos = p.cache.past_len[b] + (row - b * p.cache.seq);
+            const int b = row / p.cache.seq, pos = cached_len(p.cache.past_len, b, p.cache.max_seq) + (row - b * p.cache.seq);
             const int head = is_v ? v - s.heads - s.kv_heads : v - s.heads;
             if (pos >= p.cache.max_seq) continue;
             dst = (((size_t)b * s.kv_heads + head) * p.cache.max_seq + pos) * wide;
