@@ -4,7 +4,7 @@
 // per SM; a tile is 128 tokens x BN weight rows, K walked 64 at a time through a ring of TMA-loaded
 // operand stages (128-byte swizzle); one thread issues tcgen05.mma.kind::f16 (M 128, N BN, K 16) into
 // one of two tensor-memory accumulators, so that four read-back warps empty one tile while the next
-// is computed.  BN is 256, or 64 where 256-row tiles would leave SMs without work.  Read-back (lane =
+// is computed.  BN is 256, or 64 or 32 where larger tiles would leave SMs idle.  Read-back (lane =
 // token, 32 outputs per load), rows leave through a per-warp shared-memory block as whole pieces:
 //   PLAIN  float32
 //   GATED  a tile holds BN/2 gate rows and the matching up rows; gelu_tanh(gate) * up as bf16
