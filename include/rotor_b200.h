@@ -298,7 +298,15 @@ typedef struct rotor_b200_decoder_config {
     int32_t f32;
     float eps;            /* of every norm, the unit norm of queries and keys included */
     int32_t max_batch, max_seq, max_rows;
+    float embed_scale;    /* the residual starts as embed[id] * embed_scale */
+    const float* final_norm_b; /* [width]: the final norm is a layer norm; NULL: root mean square */
 } rotor_b200_decoder_config;
+
+/* Mixers and feed-forwards of a layer. */
+#define ROTOR_B200_MIXER_BIAS 0    /* attention over per-head keys and values, distance bias */
+#define ROTOR_B200_MIXER_LATENT 1  /* latent attention */
+#define ROTOR_B200_ACT_GELU_TANH 0
+#define ROTOR_B200_ACT_SILU 1
 
 typedef struct rotor_b200_decoder_layer {
     int32_t heads, kv_heads, dim, vdim;  /* query head h reads KV head h / (heads / kv_heads) */
@@ -314,10 +322,37 @@ typedef struct rotor_b200_decoder_layer {
     const float *norm1, *norm2;
     /* connections of the two sublayers: in [streams], out [streams], mix [from][to] */
     const float *hc1_in, *hc1_out, *hc1_mix, *hc2_in, *hc2_out, *hc2_mix;
+    /* layer norms: biases of norm1 and norm2 (both or neither; NULL: root mean square norms) */
+    const float *norm1_b, *norm2_b;
+    int32_t parallel;     /* != 0 (one stream): x + mixer(norm1(x)) + ff(norm2(x)), both of the same x */
+    int32_t window;       /* > 0: position i sees j with i - j < window */
+    const float* sinks;   /* [heads]: the softmax's denominator holds exp(sink) as well; or NULL */
+    int32_t act;          /* of the gated feed-forward */
+    /* experts > 0: the feed-forward is a mixture of `experts` gated ones of ff channels, `top` of them per token:
+     * gate_up [experts][2 ff][width], down [experts][width][ff], router [experts][width] */
+    int32_t experts, top;
+    const void* router;
+    const float* router_b;
+    /* mixer LATENT (kv_heads = 1; qkv, slopes, chunk and unit_qk unused).  Let dp = dim rounded up to 8, vp = vdim
+     * rounded up to 8, rp, kp, qp = rot_dim, kv_rank, q_rank rounded up to 16; rows and columns that rounding adds
+     * are zero.  Matrices as elsewhere (row stride rounded up to 64):
+     *   in_proj  [heads (dp + rp) queries, or qp query latents if q_rank > 0 | kp + rp, unless own_kv = 0
+     *             | heads gates, if gated][width]
+     *   uq       [heads (dp + rp)][q_rank], with q_norm [q_rank]
+     *   kv_norm  [kv_rank]
+     *   uk_uv    [heads dp key rows | heads vp value rows][kv_rank]
+     *   uk_t     [heads][kp][dim]: the key rows of a head, transposed
+     *   o        [width][heads vp]
+     *   rope     [max_seq][rot_dim / 2] cos, sin of position x frequency */
+    int32_t mixer, q_rank, kv_rank, rot_dim, gated, own_kv;
+    const void *in_proj, *uq, *uk_uv, *uk_t;
+    const float *q_norm, *kv_norm, *rope;
 } rotor_b200_decoder_layer;
 
 /* One run of a layer.  Caches: [max_batch][kv_heads][max_seq][dim rounded up to 8] (vdim for v), bf16 or
- * float32, zero-filled by the caller before first use. */
+ * float32, zero-filled by the caller before first use.  Latent attention: k_cache [max_batch][max_seq][kp + rp]
+ * holds a position's normed latent and rotated key part, v_cache is NULL; a run whose layer has own_kv = 0
+ * reads the k_cache of an earlier run and is given its pointer. */
 typedef struct rotor_b200_decoder_run {
     int32_t layer;
     void* k_cache;
@@ -336,6 +371,13 @@ int rotor_b200_decoder_create(const rotor_b200_decoder_config* cfg, const rotor_
  *    x float32 [rows][streams][n rounded up to 64], y and h [rows][n rounded up to 64]; h bf16 or float32.
  *  dense_linear: y = x w^T (float32) or, gated, gelu(x w_gate^T) (x w_up^T) in the type of x; row strides
  *    rounded up to 64; scratch float32 [rows][2 n] for gated float32 products.
+ *  norm_stage: a stage of one stream with layer norms: x = (ids ? embed[id] embed_scale : x_in + y + y2), h and
+ *    h2 the two normed rows (norm2 NULL: one).
+ *  latent_mixer: the mixer of a LATENT layer on h [rows][width rounded up to 64] (bf16 or float32), `seq` tokens
+ *    per sequence behind `past` cached ones: appends to the cache, writes y float32 [rows][width rounded up to
+ *    64].  expanded: -1 as the model chooses, 0 absorbed, 1 expanded.
+ *  experts: the routed feed-forward on h [rows][width rounded up to 64] -> y float32.
+ *    Both need rotor_b200_decoder_layer_workspace_bytes of zeroed device workspace.
  *  bias_attention: raw projections float32 [rows][q | k | v, rounded up to 64] of `seq` tokens per
  *    sequence behind past_len (device, [batch]) cached ones: appends keys and values, writes the
  *    attention rows [rows][heads vdim rounded up to 64].  Reads the head sizes and constants of
@@ -346,6 +388,15 @@ int rotor_b200_stream_stage(const int64_t* ids, const void* embed, int vocab, co
                             int streams, int n, void* h, int h_f32, void* stream);
 int rotor_b200_dense_linear(const void* w, int n, int k, const void* x, int rows, int f32, int gated, void* y, float* scratch,
                             void* stream);
+int rotor_b200_norm_stage(const int64_t* ids, const void* embed, int vocab, float embed_scale, const float* x_in, float* x_out,
+                          const float* y, const float* y2, const float* norm, const float* norm_b, const float* norm2,
+                          const float* norm2_b, float eps, int rows, int n, void* h, void* h2, int h_f32, void* stream);
+size_t rotor_b200_decoder_layer_workspace_bytes(const rotor_b200_decoder_config* cfg, const rotor_b200_decoder_layer* layer);
+int rotor_b200_latent_mixer(const rotor_b200_decoder_config* cfg, const rotor_b200_decoder_layer* layer, const void* h, int batch,
+                            int seq, int past, void* cache, int expanded, float* y, void* workspace, size_t workspace_bytes,
+                            void* stream);
+int rotor_b200_experts(const rotor_b200_decoder_config* cfg, const rotor_b200_decoder_layer* layer, const void* h, int rows,
+                       float* y, void* workspace, size_t workspace_bytes, void* stream);
 int rotor_b200_bias_attention(const rotor_b200_decoder_layer* layer, float eps, int f32, const float* qkv, int batch, int seq,
                               const int32_t* past_len, int max_seq, void* k_cache, void* v_cache, void* out, int row_kernel,
                               void* q_scratch, void* stream);

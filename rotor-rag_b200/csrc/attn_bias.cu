@@ -1,5 +1,6 @@
 // Softmax attention with a distance bias and a chunk mask, one query position at a time:
-//   score(i, j) = (q_i . k_j) scale - slope_h (i - j),   j <= i and, with chunks of C, j / C == i / C.
+//   score(i, j) = (q_i . k_j) scale - slope_h (i - j),   j <= i, with chunks of C j / C == i / C, with a window of
+// N i - j < N, and a sink per head in the softmax's denominator.
 // Used by generation steps (one token per sequence; the new key and value are normalised and appended
 // here), by short portions, by float32 runs, and by head sizes the tensor-core kernel does not take.
 //
@@ -70,12 +71,19 @@ __device__ __forceinline__ void ba_merge(const BiasAttn& p, const float* po, int
     const int total = nh * vdim;
     for (int idx = rank * nthr + tid; idx < total; idx += ns * nthr) {
         const int h = idx / vdim, c = idx - h * vdim;
-        float o, l;
+        const float sink = p.sinks ? __ldg(p.sinks + head0 + h) * 1.4426950408889634f : -INFINITY;
+        float o, l, M = sink;
         if (ns == 1) {
             o = po[h * stride + c];
             l = ml[HB + h];
+            if (p.sinks) {
+                M = fmaxf(M, ml[h]);
+                const float e = exp2f(ml[h] - M);
+                o *= e;
+                l *= e;
+            }
         } else {
-            float m[BA_MAX_SPLITS], w[BA_MAX_SPLITS], v[BA_MAX_SPLITS], M = -INFINITY;
+            float m[BA_MAX_SPLITS], w[BA_MAX_SPLITS], v[BA_MAX_SPLITS];
 #pragma unroll
             for (int k = 0; k < BA_MAX_SPLITS; ++k) {  // (all remote reads in flight together)
                 m[k] = k < ns ? ba_ld_cluster(ml + h, k) : -INFINITY;
@@ -93,6 +101,7 @@ __device__ __forceinline__ void ba_merge(const BiasAttn& p, const float* po, int
                 o += e * v[k];
             }
         }
+        if (p.sinks) l += exp2f(sink - M);
         ba_store(out + (size_t)(head0 + h) * vdim + c, o / l);
     }
     if (ns > 1)  // nobody leaves while its shared memory may still be read
@@ -121,7 +130,7 @@ __global__ void __launch_bounds__(BA_THREADS) bias_attn_rows_kernel(const __grid
     const int nh = min(HB, R - h0);                         // query heads of this CTA: hk R + h0 ..
     const int row = a.row0 + (int)blockIdx.z, b = row / p.cache.seq;
     const int pos = min(cached_len(p.cache.past_len, b, p.cache.max_seq) + (row - b * p.cache.seq), p.cache.max_seq - 1);
-    const int lo = p.chunk > 0 ? pos / p.chunk * p.chunk : 0;
+    const int lo = first_visible(pos, p.chunk, p.window);
     const int per = (pos + 1 - lo + ns - 1) / ns;
     const int t0 = lo + rank * per, t1 = min(t0 + per, pos + 1);
     const size_t head_row = ((size_t)b * s.kv_heads + hk) * p.cache.max_seq;
@@ -326,7 +335,7 @@ __global__ void __launch_bounds__(32 * NW, sizeof(T) == 2 ? 16 / NW : 1) bias_at
     const int nh = min(H, R - h0);
     const int row = a.row0 + (int)blockIdx.z, b = row / p.cache.seq;
     const int pos = min(cached_len(p.cache.past_len, b, p.cache.max_seq) + (row - b * p.cache.seq), p.cache.max_seq - 1);
-    const int lo = p.chunk > 0 ? pos / p.chunk * p.chunk : 0;
+    const int lo = first_visible(pos, p.chunk, p.window);
     const int cached = pos + (p.append ? 0 : 1) - lo;  // keys read from the cache
     // the very last warp takes the new key, the others share the cached ones
     const int strips = ns * NW - (p.append ? 1 : 0), per = (cached + strips - 1) / strips;
@@ -528,7 +537,10 @@ __global__ void __launch_bounds__(32 * NW, sizeof(T) == 2 ? 16 / NW : 1) bias_at
 }
 
 int bias_attn_reach(const BiasAttn& p) {
-    return p.chunk > 0 && p.chunk < p.cache.max_seq ? p.chunk : p.cache.max_seq;
+    int reach = p.cache.max_seq;
+    if (p.chunk > 0 && p.chunk < reach) reach = p.chunk;
+    if (p.window > 0 && p.window < reach) reach = p.window;
+    return reach;
 }
 
 template <typename T>

@@ -1,9 +1,12 @@
 // The attention of attn_bias.cu for prompts, bf16, on the fifth-generation tensor cores:
-//   score(i, j) = (q_i . k_j) scale - slope_h (i - j),   j <= i and, with chunks of C, j / C == i / C.
+//   score(i, j) = (q_i . k_j) scale - slope_h (i - j),   j <= i, j in i's chunk, i - j < window,
+// a sink per head in the softmax's denominator, and the sigmoid of a gate on each head's output.  Keys and
+// values lie in the caches, or (expanded latent attention) in rows made per head from the latents, with
+// further key columns that all heads share (template parameter DR) coming from the latent cache itself.
 //
 // CTA: 128 query rows of one KV head (row = position x query head of the group); keys 128 at a time
-// from the first key of the chunk its first position lies in up to its last position, so that keys
-// outside every row's chunk are never read.  K and V tiles arrive by TMA straight from the caches
+// from the first key its first position sees up to its last position, so that keys outside every row's
+// chunk or window are never read.  K and V tiles arrive by TMA straight from the caches
 // (heads narrower than the 64 / 128 columns of a tile are zero filled).  Both products are
 // tcgen05.mma.kind::f16 with float32 accumulators in tensor memory, scores double buffered:
 //   S = Q K^T : A = Q from shared memory (staged once), B = K tile, head dimension contiguous
@@ -24,10 +27,12 @@ namespace rb {
 
 constexpr int B5_BM = 128, B5_BN = 128, B5_THREADS = 352, B5_SOFT = 256;
 
-template <int DK, int DV>
+template <int DK, int DV, int DR>
 struct B5Cfg {
-    static constexpr int Q_BYTES = B5_BM * DK * 2, K_BYTES = B5_BN * DK * 2, V_BYTES = B5_BN * DV * 2;
-    static constexpr int SMEM = Q_BYTES + 2 * (K_BYTES + V_BYTES) + 1024 + 16384;  // (+ room for the output rows' blocks)
+    static constexpr int DQ = DK + DR;  // columns of a score
+    static constexpr int Q_BYTES = B5_BM * DQ * 2, K_BYTES = B5_BN * DQ * 2, V_BYTES = B5_BN * DV * 2;
+    static constexpr int RINGS = 2 * (K_BYTES + V_BYTES), BLOCKS = 8 * (int)T5_XPOSE_BYTES;  // (the output rows' blocks lie over the rings)
+    static constexpr int SMEM = Q_BYTES + (RINGS > BLOCKS ? RINGS : BLOCKS) + 1024;
 };
 
 struct B5Params {
@@ -35,8 +40,14 @@ struct B5Params {
     __nv_bfloat16* out;
     const int* past_len;
     const float* slopes;
+    const float* sinks;
+    const float* gate;
     unsigned* status;
-    int heads, kv_heads, kd, vdim, ld_out, seq, max_seq, chunk;
+    int heads, kv_heads, kd, vdim, ld_out, seq, max_seq, chunk, window, ld_gate;
+    int rd;                          // shared key columns of a query row, behind its kd own ones
+    // key j of KV head h in sequence b: row (b row_heads + h % row_heads) row_span + j - key0 of the K and V maps, from
+    // columns h kx_step and vx0 + h vx_step on; its shared columns: row b max_seq + j, from column rx on
+    int row_heads, row_span, key0, kx_step, vx0, vx_step, rx;
     float scale2;
 };
 
@@ -46,10 +57,12 @@ __device__ __forceinline__ float b5_exp2(float x) {
     return y;
 }
 
-template <int DK, int DV>
+template <int DK, int DV, int DR>
 __global__ void __launch_bounds__(B5_THREADS, 1)
-attn_bias_t5_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_constant__ CUtensorMap tm_v, const __grid_constant__ B5Params p) {
-    using C = B5Cfg<DK, DV>;
+attn_bias_t5_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_constant__ CUtensorMap tm_v, const __grid_constant__ CUtensorMap tm_r,
+                    const __grid_constant__ B5Params p) {
+    using C = B5Cfg<DK, DV, DR>;
+    constexpr int DQ = C::DQ;
     extern __shared__ unsigned char b5_raw[];
     __shared__ __align__(8) unsigned long long s_kfull[2], s_kempty[2], s_vfull[2], s_vempty[2], s_sfull[2], s_pfull[2], s_ofull[2],
         s_oempty[2], s_qready;
@@ -65,10 +78,10 @@ attn_bias_t5_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_const
     volatile int* abort_flag = &s_abort;
     const int s_last = min(s0 + QT, p.seq) - 1;
     const int p0 = past + s0;
-    const int kb0 = p.chunk > 0 ? p0 / p.chunk * p.chunk : 0;
+    const int kb0 = first_visible(p0, p.chunk, p.window);
     const int t_end = min(past + s_last + 1, p.max_seq);
     const int ntiles = (t_end - kb0 + B5_BN - 1) / B5_BN;
-    const int head_row = (b * p.kv_heads + hk) * p.max_seq;
+    const int head_row = (b * p.row_heads + (p.row_heads > 1 ? hk : 0)) * p.row_span - p.key0;
 
     if (threadIdx.x == 0) {
         s_abort = 0;
@@ -96,19 +109,23 @@ attn_bias_t5_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_const
 
     if (warp < 8) {
         {   // ---------------- Q tile, K-major panels of 64 columns, 128-byte swizzle
-            constexpr int QN = B5_BM * (DK / 8) / B5_SOFT;
+            constexpr int QN = B5_BM * (DQ / 8) / B5_SOFT;
+            const int qd = p.kd + p.rd;
             uint4 qv[QN];
 #pragma unroll
             for (int u = 0; u < QN; ++u) {
-                const int idx = threadIdx.x + u * B5_SOFT, r = idx / (DK / 8), c8 = idx - r * (DK / 8);
+                const int idx = threadIdx.x + u * B5_SOFT, r = idx / (DQ / 8), c8 = idx - r * (DQ / 8);
                 const int sp = r / G, s = s0 + sp, gi = r - sp * G;
+                // own key columns, then the shared ones; what lies between in a panel is zero
+                const int col = c8 < DK / 8 ? c8 * 8 : p.kd + c8 * 8 - DK;
+                const bool on = c8 < DK / 8 ? col < p.kd : col < qd;
                 qv[u] = make_uint4(0u, 0u, 0u, 0u);
-                if (sp < QT && s < p.seq && c8 * 8 < p.kd)
-                    qv[u] = __ldg(reinterpret_cast<const uint4*>(p.q + (((size_t)b * p.seq + s) * p.heads + hk * G + gi) * p.kd + c8 * 8));
+                if (sp < QT && s < p.seq && on)
+                    qv[u] = __ldg(reinterpret_cast<const uint4*>(p.q + (((size_t)b * p.seq + s) * p.heads + hk * G + gi) * qd + col));
             }
 #pragma unroll
             for (int u = 0; u < QN; ++u) {
-                const int idx = threadIdx.x + u * B5_SOFT, r = idx / (DK / 8), c8 = idx - r * (DK / 8);
+                const int idx = threadIdx.x + u * B5_SOFT, r = idx / (DQ / 8), c8 = idx - r * (DQ / 8);
                 const uint32_t dst = qbase + (uint32_t)(c8 >> 3) * 16384u + (uint32_t)(r >> 3) * 1024u + (uint32_t)(r & 7) * 128u +
                                      (uint32_t)(((c8 & 7) ^ (r & 7)) << 4);
                 asm volatile("st.shared.v4.u32 [%0], {%1, %2, %3, %4};" ::"r"(dst), "r"(qv[u].x), "r"(qv[u].y), "r"(qv[u].z), "r"(qv[u].w)
@@ -121,7 +138,7 @@ attn_bias_t5_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_const
         const int half = warp >> 2, wq = warp & 3, r = wq * 32 + lane;
         const int sp = min(r / G, QT - 1), gi = r - (r / G) * G;
         const int pos = past + min(s0 + sp, s_last);
-        const int lo = p.chunk > 0 ? pos / p.chunk * p.chunk : 0, hi = pos;  // visible keys [lo, hi]
+        const int lo = first_visible(pos, p.chunk, p.window), hi = pos;  // visible keys [lo, hi]
         const float slope2 = p.slopes ? __ldg(p.slopes + hk * G + gi) * 1.4426950408889634f : 0.f;
         const uint32_t lane_base = tmem + ((uint32_t)(wq * 32) << 16);
         float m_run = -INFINITY, l_run = 0.f, alpha_prev = 1.f;
@@ -211,7 +228,12 @@ attn_bias_t5_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_const
         l_run += s_xch[half ^ 1][r];
         if (__all_sync(0xffffffffu, ok)) {
             // rows leave through a per-warp block of the operand rings (idle: every MMA has completed)
-            const float inv = 1.0f / l_run;
+            float inv = 1.0f / l_run;
+            if (p.sinks) {
+                const float sink = __ldg(p.sinks + hk * G + gi) * 1.4426950408889634f, top = fmaxf(m_run, sink), mine = b5_exp2(m_run - top);
+                inv = mine / (l_run * mine + b5_exp2(sink - top));
+            }
+            if (p.gate) inv *= sigmoid(__ldg(p.gate + ((size_t)b * p.seq + min(s0 + sp, s_last)) * p.ld_gate + hk * G + gi));
             const uint32_t blk = kring + (uint32_t)warp * T5_XPOSE_BYTES;
             const int cpl = lane & (DV == 128 ? 7 : 3);  // 16-byte piece this lane stores
             auto dst_of = [&](int tl) -> void* {
@@ -240,7 +262,9 @@ attn_bias_t5_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_const
                 t5_bar_expect(bar, C::K_BYTES);
 #pragma unroll
                 for (int pn = 0; pn < DK / 64; ++pn)
-                    t5_tma_2d(kring + s * C::K_BYTES + pn * 16384, &tm_k, pn * 64, head_row + kb0 + j * B5_BN, bar);
+                    t5_tma_2d(kring + s * C::K_BYTES + pn * 16384, &tm_k, hk * p.kx_step + pn * 64, head_row + kb0 + j * B5_BN, bar);
+                if constexpr (DR > 0)
+                    t5_tma_2d(kring + s * C::K_BYTES + (DK / 64) * 16384, &tm_r, p.rx, b * p.max_seq + kb0 + j * B5_BN, bar);
             }
         }
     } else if (warp == 9) {
@@ -252,7 +276,7 @@ attn_bias_t5_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_const
                 t5_bar_expect(bar, C::V_BYTES);
 #pragma unroll
                 for (int pn = 0; pn < DV / 64; ++pn)
-                    t5_tma_2d(vring + s * C::V_BYTES + pn * 16384, &tm_v, pn * 64, head_row + kb0 + j * B5_BN, bar);
+                    t5_tma_2d(vring + s * C::V_BYTES + pn * 16384, &tm_v, p.vx0 + hk * p.vx_step + pn * 64, head_row + kb0 + j * B5_BN, bar);
             }
         }
     } else {
@@ -262,7 +286,7 @@ attn_bias_t5_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_const
             auto issue_s = [&](int j) {
                 const uint64_t dk = t5_desc(kring + (uint32_t)(j & 1) * C::K_BYTES);
 #pragma unroll
-                for (int k16 = 0; k16 < DK / 16; ++k16) {
+                for (int k16 = 0; k16 < DQ / 16; ++k16) {
                     const uint64_t off = (uint64_t)(((k16 >> 2) * 16384 + (k16 & 3) * 32) >> 4);
                     t5_mma_ss(tmem + (uint32_t)(j & 1) * 128u, dq + off, dk + off, idesc_s, k16 > 0);
                 }
@@ -325,16 +349,26 @@ bool bias_attn_t5_supported(const BiasAttn& p, int rows) {
            G <= B5_BM && p.ld_out % 8 == 0 && ((uintptr_t)p.out & 15) == 0 && s.kv_heads <= 65535 && rows / p.cache.seq <= 65535;
 }
 
-template <int DK, int DV>
-static int b5_launch(const BiasAttn& p, int rows, cudaStream_t st) {
-    using C = B5Cfg<DK, DV>;
+template <int DK, int DV, int DR>
+static int b5_go(const CUtensorMap& tk, const CUtensorMap& tv, const CUtensorMap& tr, B5Params& a, int batch, cudaStream_t st) {
+    using C = B5Cfg<DK, DV, DR>;
     static PerDevice<bool> once;
     if (!once.here()) {
-        RB_CUDA(cudaFuncSetAttribute(attn_bias_t5_kernel<DK, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, C::SMEM));
+        RB_CUDA(cudaFuncSetAttribute(attn_bias_t5_kernel<DK, DV, DR>, cudaFuncAttributeMaxDynamicSharedMemorySize, C::SMEM));
         once.here() = true;
     }
+    a.status = library_status_word();
+    if (!a.status) return ROTOR_B200_ERR_CUDA;
+    const int QT = B5_BM / (a.heads / a.kv_heads);
+    dim3 grid((a.seq + QT - 1) / QT, a.kv_heads, batch);
+    attn_bias_t5_kernel<DK, DV, DR><<<grid, B5_THREADS, C::SMEM, st>>>(tk, tv, tr, a);
+    return launch_status();
+}
+
+int launch_bias_attn_t5(const BiasAttn& p, int rows, cudaStream_t st) {
+    if (!bias_attn_t5_supported(p, rows)) return ROTOR_B200_ERR_SHAPE;
     const HeadShape& s = p.s;
-    const int batch = rows / p.cache.seq, G = s.heads / s.kv_heads, QT = B5_BM / G;
+    const int batch = rows / p.cache.seq;
     const size_t crows = (size_t)batch * s.kv_heads * p.cache.max_seq;
     if (crows > 0x7fffffffu) return ROTOR_B200_ERR_SHAPE;
     CUtensorMap tk, tv;
@@ -345,8 +379,7 @@ static int b5_launch(const BiasAttn& p, int rows, cudaStream_t st) {
     a.out = static_cast<__nv_bfloat16*>(p.out);
     a.past_len = p.cache.past_len;
     a.slopes = p.slopes;
-    a.status = library_status_word();
-    if (!a.status) return ROTOR_B200_ERR_CUDA;
+    a.sinks = p.sinks;
     a.heads = s.heads;
     a.kv_heads = s.kv_heads;
     a.kd = s.kd;
@@ -355,17 +388,56 @@ static int b5_launch(const BiasAttn& p, int rows, cudaStream_t st) {
     a.seq = p.cache.seq;
     a.max_seq = p.cache.max_seq;
     a.chunk = p.chunk;
+    a.window = p.window;
+    a.row_heads = s.kv_heads;
+    a.row_span = p.cache.max_seq;
     a.scale2 = p.scale * 1.4426950408889634f;
-    dim3 grid((p.cache.seq + QT - 1) / QT, s.kv_heads, batch);
-    attn_bias_t5_kernel<DK, DV><<<grid, B5_THREADS, C::SMEM, st>>>(tk, tv, a);
-    return launch_status();
+    const bool k64 = p.s.dim <= 64, v64 = p.s.vdim <= 64;
+    if (k64) return v64 ? b5_go<64, 64, 0>(tk, tv, tk, a, batch, st) : b5_go<64, 128, 0>(tk, tv, tk, a, batch, st);
+    return v64 ? b5_go<128, 64, 0>(tk, tv, tk, a, batch, st) : b5_go<128, 128, 0>(tk, tv, tk, a, batch, st);
 }
 
-int launch_bias_attn_t5(const BiasAttn& p, int rows, cudaStream_t st) {
-    if (!bias_attn_t5_supported(p, rows)) return ROTOR_B200_ERR_SHAPE;
-    const bool k64 = p.s.dim <= 64, v64 = p.s.vdim <= 64;
-    if (k64) return v64 ? b5_launch<64, 64>(p, rows, st) : b5_launch<64, 128>(p, rows, st);
-    return v64 ? b5_launch<128, 64>(p, rows, st) : b5_launch<128, 128>(p, rows, st);
+bool expanded_attn_supported(const LatentShape& s, int seq) {
+    static const bool off = getenv("ROTOR_B200_NO_TCGEN05") != nullptr;
+    return !off && seq >= 16 && s.dp <= 128 && s.rp <= 64 && s.vdim <= 128 && s.heads <= 65535;
+}
+
+int launch_expanded_attn(const ExpandedAttn& p, int batch, cudaStream_t st) {
+    const LatentShape& s = p.s;
+    const int vp = (s.vdim + 7) / 8 * 8, W = latent_row(s), ld = s.heads * (s.dp + vp);
+    if (!expanded_attn_supported(s, p.cache.seq)) return ROTOR_B200_ERR_SHAPE;
+    RB_REQUIRE(p.q && p.kv && p.out && p.cache.rows && p.cache.past_len && batch > 0 && batch <= 65535 && p.first >= 0 && p.len > 0);
+    RB_REQUIRE(p.ld_out % 8 == 0 && ((uintptr_t)p.out & 15) == 0 && (size_t)batch * p.cache.max_seq <= 0x7fffffffu);
+    CUtensorMap tk, tr;
+    if (!t5_map_bf16(&tk, p.kv, (size_t)batch * p.len, ld, ld, B5_BN) ||
+        !t5_map_bf16(&tr, p.cache.rows, (size_t)batch * p.cache.max_seq, W, W, B5_BN))
+        return ROTOR_B200_ERR_CUDA;
+    B5Params a = {};
+    a.q = p.q;
+    a.out = p.out;
+    a.past_len = p.cache.past_len;
+    a.sinks = p.sinks;
+    a.gate = p.gate;
+    a.ld_gate = p.ld_gate;
+    a.heads = a.kv_heads = s.heads;
+    a.kd = s.dp;
+    a.rd = s.rp;
+    a.vdim = vp;
+    a.ld_out = p.ld_out;
+    a.seq = p.cache.seq;
+    a.max_seq = p.cache.max_seq;
+    a.window = p.window;
+    a.row_heads = 1;
+    a.row_span = p.len;
+    a.key0 = p.first;
+    a.kx_step = s.dp;
+    a.vx0 = s.heads * s.dp;
+    a.vx_step = vp;
+    a.rx = s.kp;
+    a.scale2 = p.scale * 1.4426950408889634f;
+    const bool k64 = s.dp <= 64, v64 = vp <= 64;
+    if (k64) return v64 ? b5_go<64, 64, 64>(tk, tk, tr, a, batch, st) : b5_go<64, 128, 64>(tk, tk, tr, a, batch, st);
+    return v64 ? b5_go<128, 64, 64>(tk, tk, tr, a, batch, st) : b5_go<128, 128, 64>(tk, tk, tr, a, batch, st);
 }
 
 }  // namespace rb

@@ -7,9 +7,12 @@
 // is computed.  BN is 256, or 64 or 32 where larger tiles would leave SMs idle.  Read-back (lane =
 // token, 32 outputs per load), rows leave through a per-warp shared-memory block as whole pieces:
 //   PLAIN  float32
-//   GATED  a tile holds BN/2 gate rows and the matching up rows; gelu_tanh(gate) * up as bf16
+//   HALF   bf16, optionally times the sigmoid of a gate per token and group
+//   GATED  a tile holds BN/2 gate rows and the matching up rows; act(gate) * up as bf16
 //   QKV    the heads of the stacked q/k/v matrix: q and k divided by their root mean square, q rows
 //          out, k and v rows to the cache positions of their tokens
+// Groups (heads, sequences, experts) are more tiles of the same launch: a tile's operand and output origins
+// come from its group, or, for experts, from the table of slot runs the routing made.
 // Waits are bounded; a wait that runs out records a code in the library status word, the CTA stops
 // issuing work, frees its tensor memory and returns.  No multicast, this GPU's memory only.
 //
@@ -39,6 +42,18 @@ struct DgT5Params {
     HeadShape s;
     CacheView cache;
     __nv_bfloat16* q;
+    int act, groups, gx_col, gx_row, gw_row, gy_col, gy_row;
+    const float* head_gate;
+    int ld_head_gate;
+    const int* table;             // experts: tile count, then (expert, first slot, slots) per tile of tokens
+};
+
+// Origins of one tile.
+struct DgTile {
+    int x_row, x_col, w_row;      // operands
+    int n;                        // tile of outputs
+    int row0, rows;               // first output row; rows from there on that are this tile's own
+    int group, y_col;
 };
 
 // gelu_tanh with the fast exponential and division (their error is far below the bf16 result's)
@@ -46,6 +61,7 @@ __device__ __forceinline__ float dg_gelu(float z) {
     const float t = -1.5957691216057308f * (z + 0.044715f * z * z * z);
     return __fdividef(z, 1.0f + __expf(fminf(t, 80.f)));
 }
+__device__ __forceinline__ float dg_silu(float z) { return __fdividef(z, 1.0f + __expf(fminf(-z, 80.f))); }
 
 template <int BN, int EPI>
 __global__ void __launch_bounds__(DG5_THREADS, 1)
@@ -62,7 +78,8 @@ dense_gemm_t5_kernel(const __grid_constant__ CUtensorMap tm_a, const __grid_cons
     const uint32_t ring = (smem_u32(dg_raw) + 1023u) & ~1023u, xpose = ring + ST * C::STAGE;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     volatile int* abort_flag = &s_abort;
-    const int nk = (p.k + 63) >> 6, ntiles = p.mt * p.nt;
+    const int nk = (p.k + 63) >> 6;
+    const int mt = p.table ? __ldg(p.table) : p.mt, per_group = mt * p.nt, ntiles = per_group * p.groups;
 
     if (threadIdx.x == 0) {
         s_abort = 0;
@@ -85,11 +102,29 @@ dense_gemm_t5_kernel(const __grid_constant__ CUtensorMap tm_a, const __grid_cons
     asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
     const uint32_t tmem = s_tmem;
 
-    // tiles in groups of 16 token tiles, token tiles fastest: the CTAs of a wave share weight tiles
-    auto place = [&](int t, int& m, int& n) {
-        const int group = t / (16 * p.nt), gm = min(16, p.mt - group * 16), r = t - group * 16 * p.nt;
-        n = r / gm;
-        m = group * 16 + (r - n * gm);
+    // tiles in blocks of 16 token tiles, token tiles fastest: the CTAs of a wave share weight tiles
+    auto place = [&](int t) {
+        DgTile o;
+        o.group = t / per_group;
+        t -= o.group * per_group;
+        const int block = t / (16 * p.nt), bm = min(16, mt - block * 16), r = t - block * 16 * p.nt;
+        o.n = r / bm;
+        const int m = block * 16 + (r - o.n * bm);
+        if (p.table) {
+            const int* e = p.table + 1 + 3 * m;
+            o.group = __ldg(e);
+            o.x_row = o.row0 = __ldg(e + 1);
+            o.rows = __ldg(e + 2);
+            o.x_col = o.y_col = 0;
+        } else {
+            o.x_row = o.group * p.gx_row + m * 128;
+            o.x_col = o.group * p.gx_col;
+            o.row0 = o.group * p.gy_row + m * 128;
+            o.rows = p.rows - m * 128;
+            o.y_col = o.group * p.gy_col;
+        }
+        o.w_row = o.group * p.gw_row;
+        return o;
     };
 
     if (warp == 0) {
@@ -97,19 +132,18 @@ dense_gemm_t5_kernel(const __grid_constant__ CUtensorMap tm_a, const __grid_cons
             int it = 0;
             bool ok = true;
             for (int t = blockIdx.x; t < ntiles && ok; t += gridDim.x) {
-                int m, n;
-                place(t, m, n);
+                const DgTile at = place(t);
                 for (int kt = 0; kt < nk; ++kt, ++it) {
                     const int s = it % ST;
                     ok = t5_wait(smem_u32(&s_empty[s]), ((it / ST) & 1) ^ 1, abort_flag, p.status, 0x7a000001u);
                     if (!ok) break;
                     const uint32_t bar = smem_u32(&s_full[s]), st = ring + s * C::STAGE;
                     t5_bar_expect(bar, C::STAGE);
-                    t5_tma_2d(st, &tm_a, kt * 64, m * 128, bar);
+                    t5_tma_2d(st, &tm_a, at.x_col + kt * 64, at.x_row, bar);
 #pragma unroll
                     for (int b = 0; b < NB; ++b)
                         t5_tma_2d(st + C::A_BYTES + b * BOX * 128, &tm_b, kt * 64,
-                                  EPI == DENSE_GATED ? b * p.n + n * TN : n * TN + b * BOX, bar);
+                                  at.w_row + (EPI == DENSE_GATED ? b * p.n + at.n * TN : at.n * TN + b * BOX), bar);
                 }
             }
         }
@@ -143,13 +177,13 @@ dense_gemm_t5_kernel(const __grid_constant__ CUtensorMap tm_a, const __grid_cons
         const uint32_t stage = xpose + (uint32_t)(warp - 2) * T5_XPOSE_BYTES;
         int lt = 0;
         for (int t = blockIdx.x; t < ntiles; t += gridDim.x, ++lt) {
-            int m, n;
-            place(t, m, n);
+            const DgTile at = place(t);
+            const int n = at.n;
             const int buf = lt & 1;
             const bool good = t5_wait(smem_u32(&s_accf[buf]), (lt >> 1) & 1, abort_flag, p.status, 0x7a000004u);
             if (!__all_sync(0xffffffffu, good)) break;
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-            const int tok0 = m * 128 + wq * 32;
+            const int tok0 = at.row0 + wq * 32, tok_end = at.row0 + at.rows;
             const uint32_t tb = tmem + ((uint32_t)(wq * 32) << 16) + (uint32_t)buf * BN;
             if constexpr (EPI == DENSE_PLAIN) {
 #pragma unroll 1
@@ -159,7 +193,27 @@ dense_gemm_t5_kernel(const __grid_constant__ CUtensorMap tm_a, const __grid_cons
                     uint32_t v[32];
                     t5_ld32(tb + c * 32, v);
                     asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
-                    t5_store_rows(stage, v, p.y + (size_t)tok0 * p.ldy + col, (size_t)p.ldy * 4, tok0, p.rows, lane);
+                    t5_store_rows(stage, v, p.y + (size_t)tok0 * p.ldy + col, (size_t)p.ldy * 4, tok0, tok_end, lane);
+                }
+            } else if constexpr (EPI == DENSE_HALF) {
+                float gate = 1.f;
+                if (p.head_gate && tok0 + lane < tok_end) gate = sigmoid(__ldg(p.head_gate + (size_t)(tok0 + lane) * p.ld_head_gate + at.group));
+#pragma unroll 1
+                for (int c = 0; c < BN / 32; ++c) {
+                    const int col = n * TN + c * 32;
+                    if (col >= p.n) break;
+                    uint32_t v[32], o[16];
+                    t5_ld32(tb + c * 32, v);
+                    asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+#pragma unroll
+                    for (int i = 0; i < 16; ++i)
+                        o[i] = t5_pack(col + 2 * i < p.n ? __uint_as_float(v[2 * i]) * gate : 0.f,
+                                       col + 2 * i + 1 < p.n ? __uint_as_float(v[2 * i + 1]) * gate : 0.f);
+                    // (groups are a multiple of eight wide: 16-byte pieces past one belong to the next)
+                    const int piece = (lane & 3) * 8;
+                    t5_store_half_rows_to(stage, o, lane, [&](int tl) -> void* {
+                        return tok0 + tl < tok_end && col + piece < p.n ? p.a + (size_t)(tok0 + tl) * p.lda + at.y_col + col : nullptr;
+                    });
                 }
             } else if constexpr (EPI == DENSE_GATED) {
 #pragma unroll 1
@@ -172,12 +226,13 @@ dense_gemm_t5_kernel(const __grid_constant__ CUtensorMap tm_a, const __grid_cons
                     asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
 #pragma unroll
                     for (int i = 0; i < 16; ++i) {
-                        const float a = dg_gelu(__uint_as_float(g[2 * i])) * __uint_as_float(u[2 * i]);
-                        const float b = dg_gelu(__uint_as_float(g[2 * i + 1])) * __uint_as_float(u[2 * i + 1]);
+                        const float g0 = __uint_as_float(g[2 * i]), g1 = __uint_as_float(g[2 * i + 1]);
+                        const float a = (p.act == ACT_SILU ? dg_silu(g0) : dg_gelu(g0)) * __uint_as_float(u[2 * i]);
+                        const float b = (p.act == ACT_SILU ? dg_silu(g1) : dg_gelu(g1)) * __uint_as_float(u[2 * i + 1]);
                         o[i] = t5_pack(col + 2 * i < p.n ? a : 0.f, col + 2 * i + 1 < p.n ? b : 0.f);
                     }
                     t5_store_half_rows_to(stage, o, lane, [&](int tl) -> void* {
-                        return tok0 + tl < p.rows ? p.a + (size_t)(tok0 + tl) * p.lda + col : nullptr;
+                        return tok0 + tl < tok_end ? p.a + (size_t)(tok0 + tl) * p.lda + col : nullptr;
                     });
                 }
             } else {
@@ -250,9 +305,16 @@ bool dense_gemm_t5_supported(const DenseProduct& p, int rows) {
     if (p.f32 || rows < 1 || p.ldw % 8 || p.ldx % 8 || ((uintptr_t)p.w & 15) || ((uintptr_t)p.x & 15)) return false;
     if (p.epilogue == DENSE_PLAIN) return p.ldy % 32 == 0;
     if (p.epilogue == DENSE_GATED) return p.lda % 32 == 0;
+    if (p.epilogue == DENSE_HALF) return p.lda % 8 == 0 && (!p.groups || p.n % 8 == 0) && p.gy_col % 8 == 0 && p.gx_col % 8 == 0;
     // heads that never straddle a 64-column tile, cache rows without padding
     const HeadShape& s = p.shape;
     return (s.dim == 32 || s.dim == 64 || s.dim == 128) && s.vdim % 32 == 0 && s.kd == s.dim && s.vd == s.vdim;
+}
+
+// Tokens of all groups (of a token's choices) that tiles of 128 have to cover: tile count, at most.
+static long long dg5_token_tiles(const DenseProduct& p, int rows) {
+    if (p.route) return route_tiles((long long)rows, p.route->experts, 128);
+    return (long long)((rows + 127) / 128) * (p.groups ? p.groups : 1);
 }
 
 template <int BN, int EPI>
@@ -267,6 +329,7 @@ static int dg5_launch(const DenseProduct& p, int rows, cudaStream_t st) {
     DgT5Params a = {};
     a.status = library_status_word();
     if (!a.status) return ROTOR_B200_ERR_CUDA;
+    const int groups = p.groups ? p.groups : 1, wn = p.n * (EPI == DENSE_GATED ? 2 : 1);
     a.rows = rows;
     a.n = p.n;
     a.k = p.k;
@@ -279,51 +342,89 @@ static int dg5_launch(const DenseProduct& p, int rows, cudaStream_t st) {
     a.s = p.shape;
     a.cache = p.cache;
     a.q = p.q;
+    a.act = p.act;
+    a.groups = p.route ? 1 : groups;
+    a.gx_col = p.gx_col;
+    a.gx_row = p.gx_row;
+    a.gw_row = p.route ? wn : p.gw_row;
+    a.gy_col = p.gy_col;
+    a.gy_row = p.gy_row;
+    a.head_gate = p.head_gate;
+    a.ld_head_gate = p.ld_head_gate;
+    a.table = p.route ? p.route->table : nullptr;
+    // extents of the operands, all groups together
+    const size_t x_rows = (size_t)rows + (size_t)(groups - 1) * p.gx_row, x_cols = (size_t)p.k + (size_t)(groups - 1) * p.gx_col;
+    const size_t w_rows = p.route ? (size_t)p.route->experts * wn : (size_t)wn + (size_t)(groups - 1) * p.gw_row;
     CUtensorMap ta, tb;
-    if (!t5_map_bf16(&ta, p.x, rows, p.k, p.ldx, 128) ||
-        !t5_map_bf16(&tb, p.w, (size_t)p.n * (EPI == DENSE_GATED ? 2 : 1), p.k, p.ldw, BOX))
-        return ROTOR_B200_ERR_CUDA;
-    const int tiles = a.mt * a.nt, sms = fused_sm_count();
-    dense_gemm_t5_kernel<BN, EPI><<<tiles < sms ? tiles : sms, DG5_THREADS, C::SMEM, st>>>(ta, tb, a);
+    if (!t5_map_bf16(&ta, p.x, x_rows, x_cols, p.ldx, 128) || !t5_map_bf16(&tb, p.w, w_rows, p.k, p.ldw, BOX)) return ROTOR_B200_ERR_CUDA;
+    const long long tiles = dg5_token_tiles(p, rows) * a.nt;
+    const int sms = fused_sm_count();
+    dense_gemm_t5_kernel<BN, EPI><<<(int)(tiles < sms ? tiles : sms), DG5_THREADS, C::SMEM, st>>>(ta, tb, a);
     return launch_status();
 }
 
 int launch_dense_gemm_t5(const DenseProduct& p, int rows, cudaStream_t st) {
     if (!dense_gemm_t5_supported(p, rows)) return ROTOR_B200_ERR_SHAPE;
+    RB_REQUIRE(!p.route || (p.route->table && p.route->tile_rows == 128));
     const int tn = p.epilogue == DENSE_GATED ? 128 : 256;
-    bool wide = (long long)((rows + 127) / 128) * ((p.n + tn - 1) / tn) >= fused_sm_count();
+    const long long mt = dg5_token_tiles(p, rows);
+    bool wide = mt * ((p.n + tn - 1) / tn) >= fused_sm_count();
     if (p.epilogue == DENSE_QKV && p.shape.dim > 64) wide = true;
+    // (a few dozen rows of a narrow output: the weight stream wants as many CTAs as there are)
+    const bool narrow = mt * ((p.n + 63) / 64) * 4 < 3LL * fused_sm_count();
     switch (p.epilogue) {
         case DENSE_PLAIN:
             if (wide) return dg5_launch<256, DENSE_PLAIN>(p, rows, st);
-            // (a few dozen rows of a narrow output: the weight stream wants as many CTAs as there are)
-            return (long long)((rows + 127) / 128) * ((p.n + 63) / 64) * 4 >= 3LL * fused_sm_count() ? dg5_launch<64, DENSE_PLAIN>(p, rows, st)
-                                                                                                   : dg5_launch<32, DENSE_PLAIN>(p, rows, st);
+            return narrow ? dg5_launch<32, DENSE_PLAIN>(p, rows, st) : dg5_launch<64, DENSE_PLAIN>(p, rows, st);
+        case DENSE_HALF:
+            if (wide) return dg5_launch<256, DENSE_HALF>(p, rows, st);
+            return narrow ? dg5_launch<32, DENSE_HALF>(p, rows, st) : dg5_launch<64, DENSE_HALF>(p, rows, st);
         case DENSE_GATED: return wide ? dg5_launch<256, DENSE_GATED>(p, rows, st) : dg5_launch<64, DENSE_GATED>(p, rows, st);
         default: return wide ? dg5_launch<256, DENSE_QKV>(p, rows, st) : dg5_launch<64, DENSE_QKV>(p, rows, st);
     }
 }
 
 // ---------------------------------------------------------------------------------------
-// 64 x 64 tiles, 4 x 4 outputs per thread, K 16 at a time.
-__global__ void __launch_bounds__(256) dense_gemm_f32_kernel(const float* __restrict__ x, int ldx, const __nv_bfloat16* __restrict__ w,
-                                                             int ldw, int rows, int n, int k, float* __restrict__ y, int ldy) {
+// 64 x 64 tiles, 4 x 4 outputs per thread, K 16 at a time; grid.z: groups (experts: token tiles on grid.y, from
+// the table).
+struct DgF32 {
+    const float* x;
+    const __nv_bfloat16* w;
+    float* y;
+    int ldx, ldw, rows, n, k, ldy;
+    int gx_col, gx_row, gw_row, gy_col, gy_row;
+    const float* head_gate;
+    int ld_head_gate;
+    const int* table;
+};
+__global__ void __launch_bounds__(256) dense_gemm_f32_kernel(const __grid_constant__ DgF32 p) {
     __shared__ __align__(16) float xs[16][68], ws[16][68];
-    const int m0 = blockIdx.y * 64, n0 = blockIdx.x * 64;
+    int group = blockIdx.z, m0 = blockIdx.y * 64, end = p.rows;
+    if (p.table) {
+        if ((int)blockIdx.y >= p.table[0]) return;
+        const int* e = p.table + 1 + 3 * blockIdx.y;
+        group = e[0];
+        m0 = e[1];
+        end = m0 + e[2];
+    }
+    const float* x = p.x + (size_t)group * p.gx_row * p.ldx + (size_t)group * p.gx_col;
+    const __nv_bfloat16* w = p.w + (size_t)group * p.gw_row * p.ldw;
+    float* y = p.y + (size_t)group * p.gy_row * p.ldy + (size_t)group * p.gy_col;
+    const int n0 = blockIdx.x * 64;
     const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
     const int lr = threadIdx.x >> 2, lk = (threadIdx.x & 3) * 4;
     float acc[4][4] = {};
-    for (int k0 = 0; k0 < k; k0 += 16) {
+    for (int k0 = 0; k0 < p.k; k0 += 16) {
         float a[4] = {0.f, 0.f, 0.f, 0.f}, b[4] = {0.f, 0.f, 0.f, 0.f};
-        if (m0 + lr < rows) {
+        if (m0 + lr < end) {
 #pragma unroll
             for (int e = 0; e < 4; ++e)
-                if (k0 + lk + e < k) a[e] = x[(size_t)(m0 + lr) * ldx + k0 + lk + e];
+                if (k0 + lk + e < p.k) a[e] = x[(size_t)(m0 + lr) * p.ldx + k0 + lk + e];
         }
-        if (n0 + lr < n) {
+        if (n0 + lr < p.n) {
 #pragma unroll
             for (int e = 0; e < 4; ++e)
-                if (k0 + lk + e < k) b[e] = __bfloat162float(w[(size_t)(n0 + lr) * ldw + k0 + lk + e]);
+                if (k0 + lk + e < p.k) b[e] = __bfloat162float(w[(size_t)(n0 + lr) * p.ldw + k0 + lk + e]);
         }
         __syncthreads();
 #pragma unroll
@@ -345,18 +446,19 @@ __global__ void __launch_bounds__(256) dense_gemm_f32_kernel(const float* __rest
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
         const int r = m0 + ty * 4 + i;
-        if (r >= rows) continue;
+        if (r >= end) continue;
+        const float gate = p.head_gate ? sigmoid(p.head_gate[(size_t)r * p.ld_head_gate + group]) : 1.f;
 #pragma unroll
         for (int j = 0; j < 4; ++j)
-            if (n0 + tx * 4 + j < n) y[(size_t)r * ldy + n0 + tx * 4 + j] = acc[i][j];
+            if (n0 + tx * 4 + j < p.n) y[(size_t)r * p.ldy + n0 + tx * 4 + j] = acc[i][j] * gate;
     }
 }
 
-__global__ void __launch_bounds__(256) gate_f32_kernel(const float* __restrict__ gu, int ldgu, int rows, int ff, float* __restrict__ a, int lda) {
+__global__ void __launch_bounds__(256) gate_f32_kernel(const float* __restrict__ gu, int ldgu, int rows, int ff, int act, float* __restrict__ a, int lda) {
     const size_t total = (size_t)rows * ff;
     for (size_t i = (size_t)blockIdx.x * 256 + threadIdx.x; i < total; i += (size_t)gridDim.x * 256) {
         const int r = (int)(i / ff), c = (int)(i - (size_t)r * ff);
-        a[(size_t)r * lda + c] = gelu_tanh(gu[(size_t)r * ldgu + c]) * gu[(size_t)r * ldgu + ff + c];
+        a[(size_t)r * lda + c] = gate_act(act, gu[(size_t)r * ldgu + c]) * gu[(size_t)r * ldgu + ff + c];
     }
 }
 
@@ -364,21 +466,45 @@ __global__ void __launch_bounds__(256) gate_f32_kernel(const float* __restrict__
 int launch_dense_gemm_f32(const DenseProduct& p, int rows, float* gate_up, cudaStream_t st) {
     RB_REQUIRE(p.f32 && p.w && p.x && rows > 0 && p.epilogue != DENSE_QKV);
     const bool gated = p.epilogue == DENSE_GATED;
-    RB_REQUIRE(gated ? (gate_up && p.a) : p.y != nullptr);
-    const int n = gated ? 2 * p.n : p.n;
-    float* y = gated ? gate_up : p.y;
-    const int ldy = gated ? 2 * p.n : p.ldy;
-    for (int r0 = 0; r0 < rows; r0 += 65535 * 64) {
-        const int m = rows - r0 < 65535 * 64 ? rows - r0 : 65535 * 64;
-        dim3 grid((n + 63) / 64, (m + 63) / 64);
-        dense_gemm_f32_kernel<<<grid, 256, 0, st>>>(static_cast<const float*>(p.x) + (size_t)r0 * p.ldx, p.ldx, p.w, p.ldw, m, n, p.k,
-                                                    y + (size_t)r0 * ldy, ldy);
+    const int groups = p.groups ? p.groups : 1;
+    RB_REQUIRE(gated ? (gate_up && p.a) : (p.epilogue == DENSE_HALF ? p.a != nullptr : p.y != nullptr));
+    RB_REQUIRE(!p.route || (p.route->table && p.route->tile_rows == 64));
+    RB_REQUIRE(groups <= 65535);
+    DgF32 a = {};
+    a.x = static_cast<const float*>(p.x);
+    a.w = p.w;
+    a.ldx = p.ldx;
+    a.ldw = p.ldw;
+    a.n = gated ? 2 * p.n : p.n;
+    a.k = p.k;
+    a.y = gated ? gate_up : p.epilogue == DENSE_HALF ? static_cast<float*>(p.a) : p.y;
+    a.ldy = gated ? 2 * p.n : p.epilogue == DENSE_HALF ? p.lda : p.ldy;
+    a.gx_col = p.gx_col;
+    a.gx_row = p.gx_row;
+    a.gw_row = p.route ? a.n : p.gw_row;
+    a.gy_col = p.gy_col;
+    a.gy_row = p.gy_row;
+    a.head_gate = p.head_gate;
+    a.ld_head_gate = p.ld_head_gate;
+    const int limit = p.route ? rows : 65535 * 64;
+    for (int r0 = 0; r0 < rows; r0 += limit) {
+        const int m = rows - r0 < limit ? rows - r0 : limit;
+        const int mt = p.route ? route_tiles(m, p.route->experts, 64) : (m + 63) / 64;
+        RB_REQUIRE(mt <= 65535);
+        DgF32 b = a;
+        b.x += (size_t)r0 * p.ldx;
+        b.y += (size_t)r0 * a.ldy;
+        if (b.head_gate) b.head_gate += (size_t)r0 * p.ld_head_gate;
+        b.rows = m;
+        b.table = p.route ? p.route->table : nullptr;
+        dim3 grid((a.n + 63) / 64, mt, p.route ? 1 : groups);
+        dense_gemm_f32_kernel<<<grid, 256, 0, st>>>(b);
         int rc = launch_status();
         if (rc) return rc;
     }
     if (!gated) return ROTOR_B200_OK;
     const size_t total = (size_t)rows * p.n, blocks = (total + 255) / 256;
-    gate_f32_kernel<<<(unsigned)(blocks < 148 * 16 ? blocks : 148 * 16), 256, 0, st>>>(gate_up, 2 * p.n, rows, p.n,
+    gate_f32_kernel<<<(unsigned)(blocks < 148 * 16 ? blocks : 148 * 16), 256, 0, st>>>(gate_up, 2 * p.n, rows, p.n, p.act,
                                                                                         static_cast<float*>(p.a), p.lda);
     return launch_status();
 }

@@ -7,6 +7,11 @@
 // shares of a row are added in warp order (fixed order: repeated runs give identical bits).  A unit is
 // one 128-bit weight load per lane; loads run a batch ahead of the arithmetic, and the first batches
 // are requested before the programmatic-launch wait.
+//
+// Variants (MODE): products of two normed rows of one stage (the second a small one: a router), one product
+// per group (grid.y: heads), and a token's experts -- the gated product of each (token, choice) with the
+// expert's weights (grid.y; every CTA makes the choice itself from the router's outputs), and the weighted
+// sum of their down products as one product whose K runs over the choices.
 #include "decoder.cuh"
 
 namespace rb {
@@ -19,35 +24,67 @@ constexpr size_t DG_SMEM_MAX = 200 * 1024;
 struct DenseGemvArgs {
     DenseProduct p;
     StreamStage st;
+    Routing route;
     int has_stage, rows, slots, max_rows;
 };
+enum { GV_PLAIN = 0, GV_DUAL = 1, GV_GROUPS = 2, GV_EXPERT_UP = 3, GV_EXPERT_DOWN = 4 };
 
 // Column i (a multiple of 4) of a staged row: the two halves of a lane's eight columns sit 128 floats
 // apart, which makes both 128-bit reads of a unit free of bank conflicts.
 __device__ __forceinline__ int dg_slot(int i) { return (i & ~255) + ((i >> 2) & 1) * 128 + ((i & 255) >> 3) * 4; }
 
-template <int R, int S>
+template <int R, int S, int MODE>
 __global__ void __launch_bounds__(DG_THREADS, R <= 2 ? 2 : 1) dense_gemv_kernel(const __grid_constant__ DenseGemvArgs a) {
     const DenseProduct& p = a.p;
     extern __shared__ __align__(16) float sm[];
     __shared__ float coef[STREAMS_MAX * STREAMS_MAX + 2 * STREAMS_MAX], red[64];
-    const int kx = (p.k + 255) & ~255, steps = kx >> 8;
-    float* xs = sm;                 // [R][kx]
-    float* part = sm + R * kx;      // [local row][slot][R]
+    __shared__ int s_sel[EXPERT_TOP_MAX];
+    __shared__ float s_weight[EXPERT_TOP_MAX];
+    constexpr bool EXPERT = MODE == GV_EXPERT_UP || MODE == GV_EXPERT_DOWN;
+    const int kx = (p.k + 255) & ~255, segs = MODE == GV_EXPERT_DOWN ? a.route.top : 1, ksteps = kx >> 8, steps = ksteps * segs;
+    float* xs = sm;                 // [R][kx]; two normed rows: [2][R][kx]; several experts: [top][kx]
+    float* part = sm + (MODE == GV_DUAL ? 2 * R : R * segs) * kx;  // [local row][slot][R]
+    const int y = (int)blockIdx.y;  // group, (token, choice), token
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const bool gated = p.epilogue == DENSE_GATED;
-    const int n0 = (int)((long long)blockIdx.x * p.n / gridDim.x), n1 = (int)((long long)(blockIdx.x + 1) * p.n / gridDim.x);
+    const int n_all = MODE == GV_DUAL ? p.n + p.n2 : p.n;
+    const int n0 = (int)((long long)blockIdx.x * n_all / gridDim.x), n1 = (int)((long long)(blockIdx.x + 1) * n_all / gridDim.x);
     const int lr = (n1 - n0) * (gated ? 2 : 1);
     const int units = lr * steps, upw = max(1, (units + DG_WARPS - 1) / DG_WARPS);
     const int u0 = min(units, warp * upw), u1 = min(units, u0 + upw);
 
     // load cursor, a batch ahead of the arithmetic cursor
-    auto row_start = [&](int r) {
-        const int row = gated ? (r & 1) * p.n + n0 + (r >> 1) : n0 + r;
-        return p.w + (size_t)row * p.ldw + lane * 8;
+    auto row_start = [&](int r, int seg) {
+        int row = gated ? (r & 1) * p.n + n0 + (r >> 1) : n0 + r;
+        const __nv_bfloat16* w = p.w;
+        if constexpr (MODE == GV_DUAL)
+            if (row >= p.n) {
+                row -= p.n;
+                w = p.w2;
+            }
+        size_t at = row;
+        if constexpr (MODE == GV_GROUPS) at += (size_t)y * p.gw_row;
+        if constexpr (MODE == GV_EXPERT_UP) at += (size_t)s_sel[y % a.route.top] * 2 * p.n;
+        if constexpr (MODE == GV_EXPERT_DOWN) at += (size_t)s_sel[seg] * p.n;
+        return w + at * p.ldw + lane * 8;
     };
-    int lrow = u0 / steps, lstep = u0 - lrow * steps, lu = u0, lcol = (lstep << 8) + lane * 8;
-    const __nv_bfloat16* lp = row_start(lrow) + (lstep << 8);
+    if constexpr (EXPERT) {  // the weights depend on the router's outputs
+        pdl_wait();
+        pdl_trigger();
+        const int row = MODE == GV_EXPERT_UP ? y / a.route.top : y;
+        if (warp == 0) {
+            int sel;
+            float w;
+            route_row(a.route, row, lane, sel, w);
+            if (lane < a.route.top) {
+                s_sel[lane] = sel;
+                s_weight[lane] = w;
+            }
+        }
+        __syncthreads();
+    }
+    int lrow = u0 / steps, lstep = u0 - lrow * steps, lseg = lstep / ksteps, lu = u0, lcol = ((lstep - lseg * ksteps) << 8) + lane * 8;
+    const __nv_bfloat16* lp = row_start(lrow, lseg) + ((lstep - lseg * ksteps) << 8);
     auto fetch = [&](uint4 (&w)[DG_U]) {
 #pragma unroll
         for (int j = 0; j < DG_U; ++j) {
@@ -58,8 +95,12 @@ __global__ void __launch_bounds__(DG_THREADS, R <= 2 ? 2 : 1) dense_gemv_kernel(
             lcol += 256;
             if (++lstep == steps) {
                 lstep = 0;
+                lseg = 0;
                 lcol = lane * 8;
-                lp = row_start(++lrow);
+                lp = row_start(++lrow, 0);
+            } else if (MODE == GV_EXPERT_DOWN && lstep == (lseg + 1) * ksteps) {
+                lcol = lane * 8;
+                lp = row_start(lrow, ++lseg);
             }
         }
     };
@@ -70,8 +111,9 @@ __global__ void __launch_bounds__(DG_THREADS, R <= 2 ? 2 : 1) dense_gemv_kernel(
     for (int i = 0; i < DG_AHEAD / 8; ++i) {
         const int u = u0 + DG_U + 8 * i + (lane >> 2);
         if (u < u1) {
-            const int r = u / steps, col = ((u - r * steps) << 8) + (lane & 3) * 64;
-            if (col < p.ldw) prefetch_l2(row_start(r) - lane * 8 + col);
+            const int r = u / steps, step = u - r * steps, seg = MODE == GV_EXPERT_DOWN ? step / ksteps : 0;
+            const int col = ((step - seg * ksteps) << 8) + (lane & 3) * 64;
+            if (col < p.ldw) prefetch_l2(row_start(r, seg) - lane * 8 + col);
         }
     }
     constexpr int SG = 2;  // column groups per thread requested together
@@ -84,8 +126,10 @@ __global__ void __launch_bounds__(DG_THREADS, R <= 2 ? 2 : 1) dense_gemv_kernel(
             nw[i] = g < (a.st.ld >> 2) ? __ldg(reinterpret_cast<const float4*>(a.st.norm) + g) : make_float4(0.f, 0.f, 0.f, 0.f);
         }
     }
-    pdl_wait();
-    pdl_trigger();
+    if constexpr (!EXPERT) {
+        pdl_wait();
+        pdl_trigger();
+    }
     __syncthreads();
 
     if (a.has_stage) {
@@ -105,19 +149,41 @@ __global__ void __launch_bounds__(DG_THREADS, R <= 2 ? 2 : 1) dense_gemv_kernel(
                     float4 u = make_float4(0.f, 0.f, 0.f, 0.f);
                     if (g < n4) {
                         u = sg[i].finish(s, coef, r, g, g % gridDim.x == blockIdx.x);
-                        ss += u.x * u.x + u.y * u.y + u.z * u.z + u.w * u.w;
+                        ss += s.norm_b ? u.x + u.y + u.z + u.w : u.x * u.x + u.y * u.y + u.z * u.z + u.w * u.w;
                     }
-                    if (g < (kx >> 2)) *reinterpret_cast<float4*>(xs + r * kx + dg_slot(g << 2)) = u;
+                    if (g < (kx >> 2)) {
+                        *reinterpret_cast<float4*>(xs + r * kx + dg_slot(g << 2)) = u;
+                        if (MODE == GV_DUAL && g >= n4) *reinterpret_cast<float4*>(xs + (R + r) * kx + dg_slot(g << 2)) = u;
+                    }
                 }
             }
             ss = block_sum_alt(ss, red, k);
+            float mean = 0.f;
+            if (s.norm_b) {
+                mean = ss / (float)s.n;
+                ss = 0.f;
+                for (int g = threadIdx.x; g < n4; g += DG_THREADS)
+                    ss += squared_deviations(*reinterpret_cast<const float4*>(xs + r * kx + dg_slot(g << 2)), mean, g, s.n);
+                ss = block_sum_alt(ss, red, k);
+            }
             const float inv = 1.0f / sqrtf(ss / (float)s.n + s.eps);
             auto scale = [&](int g, const float4 w) {  // own groups
                 float4* q = reinterpret_cast<float4*>(xs + r * kx + dg_slot(g << 2));
-                float4 v = *q;
-                v = make_float4(v.x * inv * w.x, v.y * inv * w.y, v.z * inv * w.z, v.w * inv * w.w);
+                const float4 u = *q;
+                float4 v = norm_group(u, mean, inv, w, s.norm_b, g);
                 if (!p.f32) v = make_float4(round_bf16(v.x), round_bf16(v.y), round_bf16(v.z), round_bf16(v.w));
                 *q = v;
+                if constexpr (MODE == GV_DUAL) {
+                    v = norm_group(u, mean, inv, s.norm2, s.norm2_b, g);
+                    if (g % gridDim.x == blockIdx.x) {
+                        if (s.h_f32)
+                            reinterpret_cast<float4*>(static_cast<float*>(s.h2) + (size_t)r * s.ldh)[g] = v;
+                        else
+                            reinterpret_cast<uint2*>(static_cast<__nv_bfloat16*>(s.h2) + (size_t)r * s.ldh)[g] = float4_to_bf16x4(v);
+                    }
+                    if (!p.f32) v = make_float4(round_bf16(v.x), round_bf16(v.y), round_bf16(v.z), round_bf16(v.w));
+                    *reinterpret_cast<float4*>(xs + (R + r) * kx + dg_slot(g << 2)) = v;
+                }
             };
 #pragma unroll
             for (int i = 0; i < SG; ++i)
@@ -127,7 +193,15 @@ __global__ void __launch_bounds__(DG_THREADS, R <= 2 ? 2 : 1) dense_gemv_kernel(
         }
     } else {
         constexpr int XG = 4;
-        for (int r = 0; r < R; ++r)
+        const bool wide = p.f32 || p.x_raw;  // float32 rows
+        int k = 0;
+        for (int q = 0; q < R * segs; ++q) {
+            size_t at = (size_t)q * p.ldx;  // (one row: its choices)
+            if constexpr (MODE == GV_GROUPS) at += (size_t)y * p.gx_col;
+            if constexpr (MODE == GV_EXPERT_UP) at = (size_t)(y / a.route.top) * p.ldx;
+            if constexpr (MODE == GV_EXPERT_DOWN) at += (size_t)y * a.route.top * p.ldx;
+            const float gain = MODE == GV_EXPERT_DOWN ? s_weight[q] : 1.f;
+            float ss = 0.f;
             for (int g0 = threadIdx.x; g0 < (kx >> 2); g0 += XG * DG_THREADS) {
                 float4 f[XG];
 #pragma unroll
@@ -135,10 +209,10 @@ __global__ void __launch_bounds__(DG_THREADS, R <= 2 ? 2 : 1) dense_gemv_kernel(
                     const int g = g0 + i * DG_THREADS;
                     f[i] = make_float4(0.f, 0.f, 0.f, 0.f);
                     if ((g << 2) >= p.k) continue;
-                    if (p.f32)
-                        f[i] = __ldcg(reinterpret_cast<const float4*>(static_cast<const float*>(p.x) + (size_t)r * p.ldx) + g);
+                    if (wide)
+                        f[i] = __ldcg(reinterpret_cast<const float4*>(static_cast<const float*>(p.x) + at) + g);
                     else
-                        f[i] = bf16x4_to_float4(__ldcg(reinterpret_cast<const uint2*>(static_cast<const __nv_bfloat16*>(p.x) + (size_t)r * p.ldx) + g));
+                        f[i] = bf16x4_to_float4(__ldcg(reinterpret_cast<const uint2*>(static_cast<const __nv_bfloat16*>(p.x) + at) + g));
                 }
 #pragma unroll
                 for (int i = 0; i < XG; ++i) {
@@ -147,9 +221,27 @@ __global__ void __launch_bounds__(DG_THREADS, R <= 2 ? 2 : 1) dense_gemv_kernel(
                     if (c + 1 >= p.k) f[i].y = 0.f;  // (pad columns of the row may hold another product's values)
                     if (c + 2 >= p.k) f[i].z = 0.f;
                     if (c + 3 >= p.k) f[i].w = 0.f;
-                    *reinterpret_cast<float4*>(xs + r * kx + dg_slot(c)) = f[i];
+                    if constexpr (MODE == GV_EXPERT_DOWN) f[i] = make_float4(f[i].x * gain, f[i].y * gain, f[i].z * gain, f[i].w * gain);
+                    if (p.x_raw) {
+                        if (p.x_norm)
+                            ss += f[i].x * f[i].x + f[i].y * f[i].y + f[i].z * f[i].z + f[i].w * f[i].w;
+                        else if (!p.f32)
+                            f[i] = make_float4(round_bf16(f[i].x), round_bf16(f[i].y), round_bf16(f[i].z), round_bf16(f[i].w));
+                    }
+                    *reinterpret_cast<float4*>(xs + q * kx + dg_slot(c)) = f[i];
                 }
             }
+            if (!p.x_norm) continue;
+            ss = block_sum_alt(ss, red, k);
+            const float inv = 1.0f / sqrtf(ss / (float)p.k + p.x_eps);
+            for (int g = threadIdx.x; g < (kx >> 2); g += DG_THREADS) {  // own groups
+                if ((g << 2) >= p.k) continue;
+                float4* v = reinterpret_cast<float4*>(xs + q * kx + dg_slot(g << 2));
+                float4 u = norm_group(*v, 0.f, inv, p.x_norm, nullptr, g);
+                if (!p.f32) u = make_float4(round_bf16(u.x), round_bf16(u.y), round_bf16(u.z), round_bf16(u.w));
+                *v = u;
+            }
+        }
     }
     __syncthreads();
 
@@ -165,6 +257,11 @@ __global__ void __launch_bounds__(DG_THREADS, R <= 2 ? 2 : 1) dense_gemv_kernel(
             if (lane == 0) part[((size_t)crow * a.slots + slot) * R + r] = t;
             acc[r] = acc2[r] = 0.f;
         }
+    };
+    // rows of x that output row `row` (of this CTA) multiplies
+    auto operand = [&](int row) -> const float* {
+        if constexpr (MODE == GV_DUAL) return xs + (n0 + row >= p.n ? R * kx : 0);
+        return xs;
     };
     auto mac = [&](const uint4& w, const float* x) {
         const float4 wlo = bf16x4_to_float4(make_uint2(w.x, w.y)), whi = bf16x4_to_float4(make_uint2(w.z, w.w));
@@ -182,7 +279,7 @@ __global__ void __launch_bounds__(DG_THREADS, R <= 2 ? 2 : 1) dense_gemv_kernel(
         }
     };
     auto consume = [&](const uint4 (&w)[DG_U]) {
-        const float* x = xs + (cstep << 8) + lane * 4;
+        const float* x = operand(crow) + (cstep << 8) + lane * 4;
         if (cu + DG_U <= u1 && cstep + DG_U <= steps) {  // one row, the whole batch (warp-uniform)
 #pragma unroll
             for (int j = 0; j < DG_U; ++j) mac(w[j], x + (j << 8));
@@ -200,7 +297,7 @@ __global__ void __launch_bounds__(DG_THREADS, R <= 2 ? 2 : 1) dense_gemv_kernel(
 #pragma unroll
         for (int j = 0; j < DG_U; ++j) {
             if (cu < u1) {
-                mac(w[j], xs + (cstep << 8) + lane * 4);
+                mac(w[j], operand(crow) + (cstep << 8) + lane * 4);
                 ++cu;
                 if (++cstep == steps) {
                     flush();
@@ -230,85 +327,120 @@ __global__ void __launch_bounds__(DG_THREADS, R <= 2 ? 2 : 1) dense_gemv_kernel(
     };
     for (int i = threadIdx.x; i < (n1 - n0) * R; i += DG_THREADS) {
         const int r = i / (n1 - n0), o = i - r * (n1 - n0);
-        if (gated) {
-            const float v = gelu_tanh(total(2 * o, r)) * total(2 * o + 1, r);
+        auto put = [&](size_t at, float v) {
             if (p.f32)
-                static_cast<float*>(p.a)[(size_t)r * p.lda + n0 + o] = v;
+                static_cast<float*>(p.a)[at] = v;
             else
-                static_cast<__nv_bfloat16*>(p.a)[(size_t)r * p.lda + n0 + o] = __float2bfloat16_rn(v);
+                static_cast<__nv_bfloat16*>(p.a)[at] = __float2bfloat16_rn(v);
+        };
+        if (gated) {
+            const float v = gate_act(p.act, total(2 * o, r)) * total(2 * o + 1, r);
+            put((size_t)(MODE == GV_EXPERT_UP ? y : r) * p.lda + n0 + o, v);
+        } else if (MODE == GV_GROUPS) {
+            float v = total(o, r);
+            if (p.head_gate) v *= sigmoid(__ldcg(p.head_gate + (size_t)r * p.ld_head_gate + y));
+            put((size_t)r * p.lda + (size_t)y * p.gy_col + n0 + o, v);
+        } else if (MODE == GV_DUAL && n0 + o >= p.n) {
+            p.y2[(size_t)r * p.ldy2 + n0 + o - p.n] = total(o, r);
         } else {
-            p.y[(size_t)r * p.ldy + n0 + o] = total(o, r);
+            p.y[(size_t)(MODE == GV_EXPERT_DOWN ? y : r) * p.ldy + n0 + o] = total(o, r);
         }
     }
 }
 
+static int dg_mode(const DenseProduct& p) {
+    if (p.route) return p.epilogue == DENSE_GATED ? GV_EXPERT_UP : GV_EXPERT_DOWN;
+    if (p.groups) return GV_GROUPS;
+    return p.stage && p.stage->norm2 ? GV_DUAL : GV_PLAIN;
+}
+
 static size_t dg_plan(const DenseProduct& p, int rows, int* grid, int* slots) {
-    const int kx = (p.k + 255) & ~255, steps = kx / 256, pair = p.epilogue == DENSE_GATED ? 2 : 1;
-    *grid = p.n < DG_CTAS ? p.n : DG_CTAS;
-    const int lo = p.n / *grid * pair, hi = (p.n + *grid - 1) / *grid * pair;
+    const int mode = dg_mode(p), kx = (p.k + 255) & ~255, pair = p.epilogue == DENSE_GATED ? 2 : 1;
+    const int top = p.route ? p.route->top : 1, steps = kx / 256 * (mode == GV_EXPERT_DOWN ? top : 1);
+    const int n = mode == GV_DUAL ? p.n + p.n2 : p.n, planes = mode == GV_GROUPS ? p.groups : mode == GV_EXPERT_UP ? rows * top : mode == GV_EXPERT_DOWN ? rows : 1;
+    const int ctas = DG_CTAS / planes < 1 ? 1 : DG_CTAS / planes, r = p.route ? 1 : rows;
+    *grid = n < ctas ? n : ctas;
+    const int lo = n / *grid * pair, hi = (n + *grid - 1) / *grid * pair;
     const int upw = (lo * steps + DG_WARPS - 1) / DG_WARPS;
     *slots = (steps + upw - 1) / upw + 1;
-    return ((size_t)rows * kx + (size_t)hi * *slots * rows) * sizeof(float);
+    const int xrows = mode == GV_DUAL ? 2 * r : mode == GV_EXPERT_DOWN ? top : r;
+    return ((size_t)xrows * kx + (size_t)hi * *slots * r) * sizeof(float);
 }
 
 bool dense_gemv_supported(const DenseProduct& p, int rows) {
     int g, s;
+    if (p.groups > 65535 || p.epilogue == DENSE_QKV || (p.route && (p.route->top > EXPERT_TOP_MAX || p.route->top < 1))) return false;
     return rows >= 1 && rows <= DENSE_FEW_ROWS && p.n > 0 && p.k > 0 && dg_plan(p, rows, &g, &s) <= DG_SMEM_MAX;
 }
 
-template <int R, int S>
+template <int R, int S, int MODE>
 static int dg_configure() {
-    RB_CUDA(cudaFuncSetAttribute(dense_gemv_kernel<R, S>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)DG_SMEM_MAX));
+    RB_CUDA(cudaFuncSetAttribute(dense_gemv_kernel<R, S, MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)DG_SMEM_MAX));
     return ROTOR_B200_OK;
 }
 template <int R>
 static int dg_configure_all() {
     int rc;
-    if ((rc = dg_configure<R, 0>()) || (rc = dg_configure<R, 1>()) || (rc = dg_configure<R, 2>()) || (rc = dg_configure<R, 3>()) ||
-        (rc = dg_configure<R, 4>()))
+    if ((rc = dg_configure<R, 0, GV_PLAIN>()) || (rc = dg_configure<R, 1, GV_PLAIN>()) || (rc = dg_configure<R, 2, GV_PLAIN>()) ||
+        (rc = dg_configure<R, 3, GV_PLAIN>()) || (rc = dg_configure<R, 4, GV_PLAIN>()) || (rc = dg_configure<R, 1, GV_DUAL>()) ||
+        (rc = dg_configure<R, 1, GV_GROUPS>()))
         return rc;
     return ROTOR_B200_OK;
 }
 int configure_dense_gemv() {
     int rc;
-    if ((rc = dg_configure_all<1>()) || (rc = dg_configure_all<2>()) || (rc = dg_configure_all<3>()) || (rc = dg_configure_all<4>()))
+    if ((rc = dg_configure_all<1>()) || (rc = dg_configure_all<2>()) || (rc = dg_configure_all<3>()) || (rc = dg_configure_all<4>()) ||
+        (rc = dg_configure<1, 1, GV_EXPERT_UP>()) || (rc = dg_configure<1, 1, GV_EXPERT_DOWN>()))
         return rc;
     return ROTOR_B200_OK;
 }
 
 template <int R>
-static int dg_launch(const DenseGemvArgs& a, int grid, size_t smem, cudaStream_t st) {
-    const dim3 g(grid), b(DG_THREADS);
+static int dg_launch(const DenseGemvArgs& a, int mode, int grid, size_t smem, cudaStream_t st) {
+    const dim3 g(grid, mode == GV_GROUPS ? a.p.groups : 1), b(DG_THREADS);
+    if (mode == GV_GROUPS) return launch_chained(dense_gemv_kernel<R, 1, GV_GROUPS>, g, b, smem, st, 1, a);
+    if (mode == GV_DUAL) return launch_chained(dense_gemv_kernel<R, 1, GV_DUAL>, g, b, smem, st, 1, a);
     switch (a.has_stage ? a.st.streams : 1) {
-        case 1: return launch_chained(dense_gemv_kernel<R, 1>, g, b, smem, st, 1, a);
-        case 2: return launch_chained(dense_gemv_kernel<R, 2>, g, b, smem, st, 1, a);
-        case 3: return launch_chained(dense_gemv_kernel<R, 3>, g, b, smem, st, 1, a);
-        case 4: return launch_chained(dense_gemv_kernel<R, 4>, g, b, smem, st, 1, a);
-        default: return launch_chained(dense_gemv_kernel<R, 0>, g, b, smem, st, 1, a);
+        case 1: return launch_chained(dense_gemv_kernel<R, 1, GV_PLAIN>, g, b, smem, st, 1, a);
+        case 2: return launch_chained(dense_gemv_kernel<R, 2, GV_PLAIN>, g, b, smem, st, 1, a);
+        case 3: return launch_chained(dense_gemv_kernel<R, 3, GV_PLAIN>, g, b, smem, st, 1, a);
+        case 4: return launch_chained(dense_gemv_kernel<R, 4, GV_PLAIN>, g, b, smem, st, 1, a);
+        default: return launch_chained(dense_gemv_kernel<R, 0, GV_PLAIN>, g, b, smem, st, 1, a);
     }
 }
 
 int launch_dense_gemv(const DenseProduct& p, int rows, cudaStream_t st) {
     if (!dense_gemv_supported(p, rows)) return ROTOR_B200_ERR_SHAPE;
+    const int mode = dg_mode(p);
     RB_REQUIRE(p.w && p.ldw % 8 == 0 && p.ldw >= p.k && (p.stage || (p.x && p.ldx % 4 == 0)));
-    RB_REQUIRE(p.epilogue == DENSE_GATED ? p.a != nullptr : p.y != nullptr);
+    RB_REQUIRE(p.epilogue == DENSE_GATED || mode == GV_GROUPS ? p.a != nullptr : p.y != nullptr);
+    RB_REQUIRE(mode != GV_GROUPS || (p.epilogue == DENSE_HALF && p.gx_col % 4 == 0 && !p.stage));
+    RB_REQUIRE(!p.route || (p.route->logits && p.route->top <= p.route->experts && !p.stage && !p.x_norm));
+    RB_REQUIRE(!p.x_norm || p.x_raw);
     DenseGemvArgs a = {};
     a.p = p;
+    if (p.route) a.route = *p.route;
     a.rows = rows;
     a.has_stage = p.stage != nullptr;
     if (p.stage) {
         RB_REQUIRE(p.stage->streams >= 1 && p.stage->streams <= STREAMS_MAX && p.stage->n == p.k && p.stage->x_out &&
                    !p.stage->row_map);
+        RB_REQUIRE(mode != GV_DUAL || (p.stage->streams == 1 && p.stage->h2 && (p.n2 == 0 || (p.w2 && p.y2))));
+        RB_REQUIRE(!p.stage->norm2 || (p.stage->norm_b != nullptr) == (p.stage->norm2_b != nullptr));
         a.st = *p.stage;
     }
     int grid, slots;
     const size_t smem = dg_plan(p, rows, &grid, &slots);
     a.slots = slots;
+    if (mode == GV_EXPERT_UP)
+        return launch_chained(dense_gemv_kernel<1, 1, GV_EXPERT_UP>, dim3(grid, rows * p.route->top), dim3(DG_THREADS), smem, st, 1, a);
+    if (mode == GV_EXPERT_DOWN)
+        return launch_chained(dense_gemv_kernel<1, 1, GV_EXPERT_DOWN>, dim3(grid, rows), dim3(DG_THREADS), smem, st, 1, a);
     switch (rows) {
-        case 1: return dg_launch<1>(a, grid, smem, st);
-        case 2: return dg_launch<2>(a, grid, smem, st);
-        case 3: return dg_launch<3>(a, grid, smem, st);
-        default: return dg_launch<4>(a, grid, smem, st);
+        case 1: return dg_launch<1>(a, mode, grid, smem, st);
+        case 2: return dg_launch<2>(a, mode, grid, smem, st);
+        case 3: return dg_launch<3>(a, mode, grid, smem, st);
+        default: return dg_launch<4>(a, mode, grid, smem, st);
     }
 }
 

@@ -1,5 +1,5 @@
 // Row-wise stages of layer-described decoders: residual streams with hyper-connections and the
-// norm that follows (stream_stage_kernel), and the split of projection rows into normalised queries and
+// norms that follow (stream_stage_kernel), and the split of projection rows into normalised queries and
 // appended cache rows (head_finish_kernel).
 #include "decoder.cuh"
 
@@ -23,23 +23,33 @@ __global__ void __launch_bounds__(256) stream_stage_kernel(const __grid_constant
             StreamGroup<S> sg;
             sg.load(p, src, g);
             const float4 u = sg.finish(p, coef, src, g, p.x_out != nullptr);
-            ss += u.x * u.x + u.y * u.y + u.z * u.z + u.w * u.w;
+            ss += p.norm_b ? u.x + u.y + u.z + u.w : u.x * u.x + u.y * u.y + u.z * u.z + u.w * u.w;
             reinterpret_cast<float4*>(us)[g] = u;
         }
         if (!p.h) continue;
+        float mean = 0.f;
         ss = block_sum_alt(ss, red, k);
+        if (p.norm_b) {  // own groups of us
+            mean = ss / (float)p.n;
+            ss = 0.f;
+            for (int g = threadIdx.x; g < n4; g += blockDim.x) ss += squared_deviations(reinterpret_cast<const float4*>(us)[g], mean, g, p.n);
+            ss = block_sum_alt(ss, red, k);
+        }
         const float inv = 1.0f / sqrtf(ss / (float)p.n + p.eps);
-        for (int g = threadIdx.x; g < (p.ldh >> 2); g += blockDim.x) {  // own groups of us, zeros behind them
-            float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-            if (g < n4) {
-                v = reinterpret_cast<const float4*>(us)[g];
-                const float4 w = __ldg(reinterpret_cast<const float4*>(p.norm) + g);
-                v = make_float4(v.x * inv * w.x, v.y * inv * w.y, v.z * inv * w.z, v.w * inv * w.w);
-            }
+        auto store = [&](void* h, int g, const float4 v) {
             if (p.h_f32)
-                reinterpret_cast<float4*>(static_cast<float*>(p.h) + (size_t)r * p.ldh)[g] = v;
+                reinterpret_cast<float4*>(static_cast<float*>(h) + (size_t)r * p.ldh)[g] = v;
             else
-                reinterpret_cast<uint2*>(static_cast<__nv_bfloat16*>(p.h) + (size_t)r * p.ldh)[g] = float4_to_bf16x4(v);
+                reinterpret_cast<uint2*>(static_cast<__nv_bfloat16*>(h) + (size_t)r * p.ldh)[g] = float4_to_bf16x4(v);
+        };
+        for (int g = threadIdx.x; g < (p.ldh >> 2); g += blockDim.x) {  // own groups of us, zeros behind them
+            float4 v = make_float4(0.f, 0.f, 0.f, 0.f), u = v;
+            if (g < n4) {
+                u = reinterpret_cast<const float4*>(us)[g];
+                v = norm_group(u, mean, inv, p.norm, p.norm_b, g);
+            }
+            store(p.h, g, v);
+            if (p.norm2) store(p.h2, g, g < n4 ? norm_group(u, mean, inv, p.norm2, p.norm2_b, g) : v);
         }
     }
 }
@@ -48,6 +58,7 @@ int launch_stream_stage(const StreamStage& p, int rows, cudaStream_t st) {
     RB_REQUIRE(rows > 0 && p.streams >= 1 && p.streams <= STREAMS_MAX && p.ld % 4 == 0 && p.ldh % 4 == 0);
     const size_t smem = (size_t)p.ld * sizeof(float);
     if (smem > 40 * 1024) return ROTOR_B200_ERR_SHAPE;
+    RB_REQUIRE(!p.norm2 || (p.h && p.h2 && (p.norm_b != nullptr) == (p.norm2_b != nullptr)));
     const int threads = p.ld >= 1024 ? 256 : (p.ld >= 256 ? 128 : 64);
     const int per_sm = 2048 / threads;
     dim3 grid(rows < 148 * per_sm ? rows : 148 * per_sm), block(threads);

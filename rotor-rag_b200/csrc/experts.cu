@@ -1,0 +1,108 @@
+// Routing of many tokens to their experts: choice and weights, slots grouped by expert, the table of token
+// tiles the expert products walk, and the copy of the rows into their slots.  (Up to DENSE_FEW_ROWS tokens
+// need none of this: the matrix-vector products choose for themselves.)
+#include "decoder.cuh"
+
+namespace rb {
+
+// One warp per row: choices, weights, and how many rows each expert gets.
+__global__ void __launch_bounds__(256) route_choose_kernel(const __grid_constant__ Routing r, int rows) {
+    __shared__ int hist[EXPERTS_MAX];
+    for (int e = threadIdx.x; e < r.experts; e += blockDim.x) hist[e] = 0;
+    pdl_wait();
+    pdl_trigger();
+    __syncthreads();
+    const int lane = threadIdx.x & 31, per = blockDim.x >> 5;
+    for (int row = blockIdx.x * per + (threadIdx.x >> 5); row < rows; row += gridDim.x * per) {
+        int sel;
+        float w;
+        route_row(r, row, lane, sel, w);
+        if (lane < r.top) {
+            r.chosen[(size_t)row * r.top + lane] = sel;
+            r.weight[(size_t)row * r.top + lane] = w;
+            atomicAdd(&hist[sel], 1);
+        }
+    }
+    __syncthreads();
+    for (int e = threadIdx.x; e < r.experts; e += blockDim.x)
+        if (hist[e]) atomicAdd(&r.counts[e], hist[e]);
+}
+
+// One CTA of EXPERTS_MAX threads: first slot of every expert, the tile table; counts are zeroed for the next call.
+__global__ void __launch_bounds__(EXPERTS_MAX) route_table_kernel(const __grid_constant__ Routing r) {
+    __shared__ int2 warp_sums[32];
+    pdl_wait();
+    pdl_trigger();
+    const int e = threadIdx.x, lane = e & 31, warp = e >> 5;
+    const int n = e < r.experts ? r.counts[e] : 0, tiles = (n + r.tile_rows - 1) / r.tile_rows;
+    int2 s = make_int2(n, tiles);  // inclusive sums
+    auto scan = [&]() {
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+            const int a = __shfl_up_sync(0xffffffffu, s.x, o), b = __shfl_up_sync(0xffffffffu, s.y, o);
+            if (lane >= o) {
+                s.x += a;
+                s.y += b;
+            }
+        }
+    };
+    scan();
+    if (lane == 31) warp_sums[warp] = s;
+    __syncthreads();
+    const int2 own = s;
+    if (warp == 0) {
+        s = warp_sums[lane];
+        scan();
+        warp_sums[lane] = s;
+    }
+    __syncthreads();
+    int first = own.x - n, tile = own.y - tiles;
+    if (warp > 0) {
+        first += warp_sums[warp - 1].x;
+        tile += warp_sums[warp - 1].y;
+    }
+    if (e < r.experts) {
+        r.cursor[e] = first;
+        r.counts[e] = 0;
+        for (int t = 0; t < tiles; ++t) {
+            int* out = r.table + 1 + 3 * (tile + t);
+            out[0] = e;
+            out[1] = first + t * r.tile_rows;
+            out[2] = min(r.tile_rows, n - t * r.tile_rows);
+        }
+    }
+    if (e == 0) r.table[0] = warp_sums[31].y;
+}
+
+// One warp per (row, choice): takes the expert's next slot and copies the row there.
+__global__ void __launch_bounds__(256) route_scatter_kernel(const __grid_constant__ Routing r, int pairs, const uint4* x, int pieces, uint4* permuted) {
+    pdl_wait();
+    pdl_trigger();
+    const int lane = threadIdx.x & 31, per = blockDim.x >> 5;
+    for (int i = blockIdx.x * per + (threadIdx.x >> 5); i < pairs; i += gridDim.x * per) {
+        int slot = 0;
+        if (lane == 0) {
+            slot = atomicAdd(&r.cursor[r.chosen[i]], 1);
+            r.slot_of[i] = slot;
+        }
+        slot = __shfl_sync(0xffffffffu, slot, 0);
+        const uint4* src = x + (size_t)(i / r.top) * pieces;
+        uint4* dst = permuted + (size_t)slot * pieces;
+        for (int c = lane; c < pieces; c += 32) dst[c] = __ldg(src + c);
+    }
+}
+
+int launch_route(const Routing& r, int rows, const void* x, size_t row_bytes, void* permuted, cudaStream_t st) {
+    RB_REQUIRE(r.logits && r.slot_of && r.weight && r.chosen && r.counts && r.cursor && r.table && x && permuted && rows > 0);
+    RB_REQUIRE(r.experts >= 1 && r.experts <= EXPERTS_MAX && r.top >= 1 && r.top <= r.experts && r.top <= EXPERT_TOP_MAX);
+    RB_REQUIRE(row_bytes % 16 == 0 && (long long)rows * r.top < 0x7fffffffLL);
+    const int pairs = rows * r.top, most = 148 * 8;
+    int rc = launch_chained(route_choose_kernel, dim3((rows + 7) / 8 < most ? (rows + 7) / 8 : most), dim3(256), 0, st, 1, r, rows);
+    if (!rc) rc = launch_chained(route_table_kernel, dim3(1), dim3(EXPERTS_MAX), 0, st, 1, r);
+    if (!rc)
+        rc = launch_chained(route_scatter_kernel, dim3((pairs + 7) / 8 < most ? (pairs + 7) / 8 : most), dim3(256), 0, st, 1, r, pairs,
+                            static_cast<const uint4*>(x), (int)(row_bytes / 16), static_cast<uint4*>(permuted));
+    return rc;
+}
+
+}  // namespace rb

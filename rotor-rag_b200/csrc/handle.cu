@@ -69,6 +69,7 @@ int rotor_b200_model_forward(void* handle, const int64_t* ids, int batch, int se
     RB_REQUIRE(logits_mode == ROTOR_B200_LOGITS_NONE || logits);
     cudaStream_t st = as_stream(stream);
     RB_TRY(launch_set_pos(m->c.d_pos, m->c.max_batch, past_len, nullptr, st));
+    m->past = past_len;
     RB_TRY(forward_family(*m, (const long long*)ids, batch, seq, logits_mode, logits, (long long*)next_ids, st));
     m->pos = past_len + seq;
     return launch_status();
@@ -83,6 +84,7 @@ int rotor_b200_model_forward_rows(void* handle, const int64_t* ids, int batch, i
     for (int i = 0; i < nrows; ++i) RB_REQUIRE(rows[i] >= 0 && rows[i] < batch * seq);
     cudaStream_t st = as_stream(stream);
     RB_TRY(launch_set_pos(m->c.d_pos, m->c.max_batch, past_len, nullptr, st));
+    m->past = past_len;
     const int32_t none = 0;
     m->want = nrows ? rows : &none;
     m->nwant = nrows;
@@ -123,6 +125,7 @@ int rotor_b200_model_forward_ragged(void* handle, const int64_t* ids, int batch,
     for (int b = 0; b < batch; ++b) RB_REQUIRE(lens[b] >= 1 && lens[b] <= seq);
     cudaStream_t st = as_stream(stream);
     RB_TRY(launch_set_pos(m->c.d_pos, m->c.max_batch, 0, nullptr, st));
+    m->past = 0;
     m->last_of = lens;
     const int rc = forward_family(*m, (const long long*)ids, batch, seq, logits_mode, logits, (long long*)next_ids, st);
     m->last_of = nullptr;

@@ -95,6 +95,7 @@ struct Model {
     bool no_fused;        // comparison aid: unfused stages in every forward
     const int32_t* want;  // host, during a forward of selected rows: rows whose logits are wanted
     int nwant;
+    int past;             // during a forward of many tokens: their sequences' cached length
 };
 
 struct Carve {

@@ -124,7 +124,12 @@ class DecoderConfig(C.Structure):
     """rotor_b200_decoder_config"""
     _fields_ = [("vocab_size", C.c_int32), ("width", C.c_int32), ("streams", C.c_int32), ("n_layers", C.c_int32),
                 ("n_runs", C.c_int32), ("f32", C.c_int32), ("eps", C.c_float),
-                ("max_batch", C.c_int32), ("max_seq", C.c_int32), ("max_rows", C.c_int32)]
+                ("max_batch", C.c_int32), ("max_seq", C.c_int32), ("max_rows", C.c_int32),
+                ("embed_scale", _f), ("final_norm_b", _p)]
+
+
+MIXER_BIAS, MIXER_LATENT = 0, 1
+ACT_GELU_TANH, ACT_SILU = 0, 1
 
 
 class DecoderLayer(C.Structure):
@@ -132,7 +137,12 @@ class DecoderLayer(C.Structure):
     _fields_ = [("heads", C.c_int32), ("kv_heads", C.c_int32), ("dim", C.c_int32), ("vdim", C.c_int32),
                 ("unit_qk", C.c_int32), ("chunk", C.c_int32), ("ff", C.c_int32), ("scale", _f), ("slopes", _p),
                 ("qkv", _p), ("o", _p), ("gate_up", _p), ("down", _p), ("norm1", _p), ("norm2", _p),
-                ("hc1_in", _p), ("hc1_out", _p), ("hc1_mix", _p), ("hc2_in", _p), ("hc2_out", _p), ("hc2_mix", _p)]
+                ("hc1_in", _p), ("hc1_out", _p), ("hc1_mix", _p), ("hc2_in", _p), ("hc2_out", _p), ("hc2_mix", _p),
+                ("norm1_b", _p), ("norm2_b", _p), ("parallel", C.c_int32), ("window", C.c_int32), ("sinks", _p),
+                ("act", C.c_int32), ("experts", C.c_int32), ("top", C.c_int32), ("router", _p), ("router_b", _p),
+                ("mixer", C.c_int32), ("q_rank", C.c_int32), ("kv_rank", C.c_int32), ("rot_dim", C.c_int32),
+                ("gated", C.c_int32), ("own_kv", C.c_int32), ("in_proj", _p), ("uq", _p), ("uk_uv", _p), ("uk_t", _p),
+                ("q_norm", _p), ("kv_norm", _p), ("rope", _p)]
 
 
 class DecoderRun(C.Structure):
@@ -148,6 +158,10 @@ _SIGNATURES.update({
     "rotor_b200_decoder_create": (_i, [_dcp, _dlp, _drp, _p, _p, _p, _p, _sz, C.POINTER(_p)]),
     "rotor_b200_stream_stage": (_i, [_p, _p, _i, _p, _p, _p, _p, _p, _p, _p, _f, _i, _i, _i, _p, _i, _p]),
     "rotor_b200_dense_linear": (_i, [_p, _i, _i, _p, _i, _i, _i, _p, _p, _p]),
+    "rotor_b200_norm_stage": (_i, [_p, _p, _i, _f, _p, _p, _p, _p, _p, _p, _p, _p, _f, _i, _i, _p, _p, _i, _p]),
+    "rotor_b200_decoder_layer_workspace_bytes": (_sz, [_dcp, _dlp]),
+    "rotor_b200_latent_mixer": (_i, [_dcp, _dlp, _p, _i, _i, _i, _p, _i, _p, _p, _sz, _p]),
+    "rotor_b200_experts": (_i, [_dcp, _dlp, _p, _i, _p, _p, _sz, _p]),
     "rotor_b200_bias_attention": (_i, [_dlp, _f, _i, _p, _i, _i, _p, _i, _p, _p, _p, _i, _p, _p]),
 })
 

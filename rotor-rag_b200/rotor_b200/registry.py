@@ -44,6 +44,12 @@ def _likerax(model_dir, config, dtype, **kw):
     return load_likerax_model(model_dir, config, dtype=dtype, **kw)
 
 
+@register("Miborax")
+def _miborax(model_dir, config, dtype, **kw):
+    from .miborax import load_miborax_model
+    return load_miborax_model(model_dir, config, dtype=dtype, **kw)
+
+
 def load_model(model_dir, dtype: str = "bfloat16", **kw):
     model_dir = Path(model_dir)
     with open(model_dir / "config.json") as f:

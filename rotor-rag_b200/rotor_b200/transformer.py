@@ -175,6 +175,8 @@ class KVCache:
 
     def __getitem__(self, key):
         buf = {"k": self.owner.k_cache, "v": self.owner.v_cache}[key]
+        if buf is None:
+            raise KeyError(key)   # (latent attention: one row per position, under "k")
         return buf[: self.batch, :, : self.length, :].cpu().numpy()
 
     def __len__(self):
