@@ -156,7 +156,7 @@ struct LatentRun {
         const int n = min(tile, t1 - k0), pieces = W / PIECE;
         for (int i = threadIdx.x; i < tile * pieces; i += LA_THREADS) {
             const int j = i / pieces, c = i - j * pieces;
-            if (k0 + j == skip) continue;
+            if (k0 + j == skip && j < n) continue;
             const int bytes = j < n ? 16 : 0;
             const T* src = rows + (size_t)(j < n ? k0 + j : k0) * W + c * PIECE;
             asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(la_smem(dst + (size_t)j * stride + c * PIECE)), "l"(src), "r"(bytes)
