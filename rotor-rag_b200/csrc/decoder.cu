@@ -54,6 +54,7 @@ struct DecoderStack {
     void *q_abs, *o_lat;         // absorbed queries, weighted latents (abs_rows of them)
     __nv_bfloat16* kv;           // expanded keys and values [kv_rows]
     int abs_rows, kv_rows;
+    bool absorb_all;             // workspace for prompts in the absorbed form too
     // experts
     float* logits;               // router outputs [rows][lde]
     void *perm, *slots;          // rows by slot; their outputs
@@ -146,7 +147,7 @@ static void carve_decoder(Model& m, DecoderStack& d, const rotor_b200_decoder_la
         size_t qkv = 0, q = 0, attn = 0, act = 0, gu = 0, q_raw = 0, cq = 0, lq = 0, abs = 0, lat = 0, kv = 0, lde = 0, slots = 0, experts = 0, top = 0;
     } w;
     auto widen = [](size_t& v, size_t n) { v = n > v ? n : v; };
-    bool parallel = false, absorb_all = false;
+    bool parallel = false, absorb_all = d.absorb_all;
     for (int l = 0; l < c.n_layers; ++l) {
         const rotor_b200_decoder_layer& L = layers[l];
         parallel |= L.parallel != 0;
@@ -652,6 +653,7 @@ size_t rotor_b200_decoder_workspace_bytes(const rotor_b200_decoder_config* cfg, 
     memset(&m, 0, sizeof(m));
     DecoderStack d;
     d.cfg = *cfg;
+    d.absorb_all = false;
     size_t total = 0;
     carve_decoder(m, d, layers, nullptr, &total);
     return total;
@@ -684,6 +686,7 @@ int rotor_b200_decoder_create(const rotor_b200_decoder_config* cfg, const rotor_
     m->decoder = d;
     m->no_fused = getenv("ROTOR_B200_NO_FUSED_STEP") != nullptr;
     d->cfg = *cfg;
+    d->absorb_all = false;
     d->layers.assign(layers, layers + cfg->n_layers);
     d->runs.assign(runs, runs + cfg->n_runs);
     d->embed = static_cast<const __nv_bfloat16*>(embed);
@@ -806,6 +809,7 @@ struct OneLayer {
         RB_REQUIRE(cfg && layer && workspace && ((uintptr_t)workspace & 255) == 0 && cfg->n_layers == 1);
         RB_TRY(check_decoder(*cfg, layer, nullptr));
         d.cfg = *cfg;
+        d.absorb_all = true;
         m.decoder = &d;
         m.no_fused = getenv("ROTOR_B200_NO_FUSED_STEP") != nullptr;
         size_t total = 0;
@@ -815,7 +819,15 @@ struct OneLayer {
 };
 
 size_t rotor_b200_decoder_layer_workspace_bytes(const rotor_b200_decoder_config* cfg, const rotor_b200_decoder_layer* layer) {
-    return cfg && cfg->n_layers == 1 ? rotor_b200_decoder_workspace_bytes(cfg, layer) : 0;
+    if (!cfg || !layer || cfg->n_layers != 1 || check_decoder(*cfg, layer, nullptr)) return 0;
+    Model m;
+    memset(&m, 0, sizeof(m));
+    DecoderStack d;
+    d.cfg = *cfg;
+    d.absorb_all = true;
+    size_t total = 0;
+    carve_decoder(m, d, layer, nullptr, &total);
+    return total;
 }
 
 int rotor_b200_latent_mixer(const rotor_b200_decoder_config* cfg, const rotor_b200_decoder_layer* layer, const void* h, int batch,
