@@ -34,6 +34,7 @@ One JSON line is printed by rank 0:
 --impl reference times the reference itself on the host cores (its installed copy under baseline/_ref,
 through its own TextGenerator.generate; the port stands in where the copy is absent).
 --workload likerax times the Likerax design beside the ternary model at equal sizes.
+--workload miborax times the Miborax design beside Likerax at equal sizes.
 --workload / --only select one section alone (profiling aids; they print their own line).
 """
 import argparse
@@ -955,18 +956,16 @@ def likerax_kernels(torch, abi, cfg, B, S, chunk, streams=2):
     return out
 
 
-def run_likerax(args):
-    """--workload likerax: prefill and decode throughput of the Likerax design beside the ternary model at
-    equal sizes (random weights; the ternary model's float work per token is the same, its weights are 2 bits)."""
+def run_designs(args, metric, shapes, families, sublayers):
+    """One line: prefill and decode throughput of two designs at equal sizes, random weights.  shapes: name ->
+    (sizes, layers, sequences); families: name -> builder(sizes, model keywords); sublayers: what else to time."""
     import torch
-    from rotor_b200 import abi, semantics
-    from rotor_b200.synth import XL_TP, random_model_on_device
+    from rotor_b200 import abi
     torch.cuda.set_device(0)
     barrier = torch.cuda.synchronize
     K, W = args.steps, max(args.warmup, 3)
     prompt_len, S = XL_PROMPT_LEN, args.seq or 2048
-    shapes = {"2b": (dict(CFG_2B), args.layers or 6, args.batch or 8), "xl": (dict(XL_TP), min(args.layers or 2, 4), args.batch or 2)}
-    line = {"metric": "Likerax prefill and decode tokens/s beside the ternary model at equal size", "unit": UNIT, "n_gpus": 1,
+    line = {"metric": metric, "unit": UNIT, "n_gpus": 1,
             "steps": K, "warmup": W, "higher_is_better": True, "data": "synthetic", "dtype": "bf16 (float32 residual, scores, norms)",
             "shapes": {}}
     before = abi.lib.rotor_b200_launch_count()
@@ -974,14 +973,12 @@ def run_likerax(args):
         if args.only in shapes and args.only != name:
             continue
         cfg["n_layers"] = layers
-        rec = {"config": dict(cfg, streams=2, chunk=args.chunk, prefill=f"{B} x {S}", decode=f"after {prompt_len} tokens")}
-        for family in ("likerax", "bitnet"):
+        rec = {"config": dict(cfg, prefill=f"{B} x {S}", decode=f"after {prompt_len} tokens")}
+        for family, make in families.items():
             if args.family not in ("both", family):
                 continue
             max_seq = max(S, prompt_len + 1 + W + K + 8)
-            kw = dict(max_seq=max_seq, max_batch=B, max_rows=B * S)
-            model = likerax_random(cfg, layers, args.chunk, **kw) if family == "likerax" else \
-                random_model_on_device(cfg, seed=3, semantics=semantics.BASELINE, **kw)
+            model = make(cfg, dict(max_seq=max_seq, max_batch=B, max_rows=B * S))
             r = {}
             if args.phase in ("both", "prefill"):
                 r["prefill"] = time_prefill(torch, abi, model, cfg["vocab_size"], B, S, 5, 3)
@@ -999,11 +996,132 @@ def run_likerax(args):
             h = None
             torch.cuda.empty_cache()
         if args.family == "both" and args.phase == "both":
-            rec["likerax_kernels"] = likerax_kernels(torch, abi, cfg, B, S, args.chunk)
+            rec.update(sublayers(torch, abi, cfg, B, S))
             torch.cuda.empty_cache()
         line["shapes"][name] = rec
     line["gpu_launches"] = int(abi.lib.rotor_b200_launch_count() - before)
     print(json.dumps(line), flush=True)
+
+
+def run_likerax(args):
+    """--workload likerax: prefill and decode throughput of the Likerax design beside the ternary model at
+    equal sizes (random weights; the ternary model's float work per token is the same, its weights are 2 bits)."""
+    from rotor_b200 import semantics
+    from rotor_b200.synth import XL_TP, random_model_on_device
+    extra = dict(streams=2, chunk=args.chunk)
+    shapes = {"2b": (dict(CFG_2B, **extra), args.layers or 6, args.batch or 8),
+              "xl": (dict(XL_TP, **extra), min(args.layers or 2, 4), args.batch or 2)}
+    run_designs(args, "Likerax prefill and decode tokens/s beside the ternary model at equal size", shapes,
+                {"likerax": lambda cfg, kw: likerax_random(cfg, cfg["n_layers"], args.chunk, **kw),
+                 "bitnet": lambda cfg, kw: random_model_on_device({k: v for k, v in cfg.items() if k not in extra}, seed=3,
+                                                                  semantics=semantics.BASELINE, **kw)},
+                lambda torch, abi, cfg, B, S: {"likerax_kernels": likerax_kernels(torch, abi, cfg, B, S, args.chunk)})
+
+
+# Sizes of a latent-attention mixture of experts as such models are built; d_ff is what a token's experts add up to.
+MIBORAX_16H = dict(vocab_size=102400, d_model=2048, n_heads=16, n_kv_heads=16, d_ff=6 * 1408, dim=128, rot=64, vdim=128, kv_rank=512,
+                   q_rank=1536, window=1024, experts=64, top=6, expert_ff=1408)
+MIBORAX_40H = dict(vocab_size=102400, d_model=5120, n_heads=40, n_kv_heads=40, d_ff=6 * 1536, dim=128, rot=64, vdim=128, kv_rank=512,
+                   q_rank=1536, window=1024, experts=64, top=6, expert_ff=1536)
+
+
+def miborax_layers(cfg, layers, seed=0):
+    """Layer specs of the design, random weights: a windowed layer, one that borrows its cache, and a layer over the whole
+    past, in turn."""
+    import torch
+    from rotor_b200.decoder_model import Experts, Latent, LayerSpec
+    g = torch.Generator(device="cuda")
+    g.manual_seed(seed)
+    d, h, ff, n = cfg["d_model"], cfg["n_heads"], cfg["expert_ff"], cfg["experts"]
+    mat = lambda o, i: (torch.randn((o, i), generator=g, device="cuda") / i ** 0.5).to(torch.bfloat16)
+    qd, rank, rot = cfg["dim"] + cfg["rot"], cfg["kv_rank"], cfg["rot"]
+    one, zero = torch.ones(d), torch.zeros(d)
+    specs = []
+    for i in range(layers):
+        full, lent = i % 3 == 2, i % 3 == 1
+        a = Latent(rank, rot, 10000.0, mat(h * cfg["dim"], rank), mat(h * cfg["vdim"], rank))
+        if lent:
+            a.kv_from = i - 1
+        else:
+            a.dkv, a.kv_norm = mat(rank + rot, d), torch.ones(rank)
+        if full:
+            a.dq, a.q_norm, a.uq, a.gate = mat(cfg["q_rank"], d), torch.ones(cfg["q_rank"]), mat(h * qd, cfg["q_rank"]), mat(h, d)
+        each = lambda o, k: [mat(o, k) for _ in range(n)]
+        specs.append(LayerSpec(h, 1, cfg["dim"], cfg["vdim"], qd ** -0.5, None if full else mat(h * qd, d), None, None, mat(d, h * cfg["vdim"]),
+                               one, window=0 if full else cfg["window"], sinks=torch.zeros(h), act="silu", norm1_b=zero, norm2=one, norm2_b=zero,
+                               parallel=True, latent=a,
+                               experts=Experts(cfg["top"], mat(n, d), each(ff, d), each(ff, d), each(d, ff), bias=torch.zeros(n))))
+    return specs, mat(cfg["vocab_size"], d), one, zero
+
+
+def miborax_random(cfg, layers, seed=0, **kw):
+    from rotor_b200.decoder_model import DecoderModel
+    specs, embed, one, zero = miborax_layers(cfg, layers, seed)
+    return DecoderModel(specs, range(layers), embed, None, one, final_norm_b=zero, eps=1e-5, embed_scale=cfg["d_model"] ** 0.5, **kw)
+
+
+def miborax_sublayers(torch, abi, cfg, B, S):
+    """The mixers and the experts of one layer alone: prompts of B x S tokens, and one token of 1 and B sequences."""
+    import ctypes as C
+    lib = abi.lib
+    with open(os.path.join(ROOT, "MEASURED_PEAKS.json")) as f:
+        peaks = json.load(f)
+    hbm, tflops = peaks["hbm_gbs"] * 1e9, peaks["bf16_tflops"] * 1e12
+    d, h, qd, rank, row = cfg["d_model"], cfg["n_heads"], cfg["dim"] + cfg["rot"], cfg["kv_rank"], cfg["kv_rank"] + cfg["rot"]
+    n, top, ff, W = cfg["experts"], cfg["top"], cfg["expert_ff"], cfg["window"]
+    model = miborax_random(cfg, 3, max_seq=S + 64, max_batch=B, max_rows=B * S)
+    hd = model._ensure_handle(B, S, S + 1)
+    out = {}
+
+    def record(name, sec, nbytes, flops):
+        """Roofline: the slower of the bytes at the measured copy rate and the multiplications at the measured bf16 rate."""
+        bound = max(nbytes / hbm, flops / tflops)
+        out[name] = {"us": sec * 1e6, "bytes": nbytes, "flops": flops, "roofline_us": bound * 1e6, "frac_of_roofline": bound / sec}
+
+    one = abi.DecoderConfig.from_buffer_copy(hd.cfg)
+    one.n_layers = one.n_runs = 1
+    x = torch.randn((B * S, d), device="cuda").to(torch.bfloat16)
+    y = torch.empty((B * S, d), device="cuda")
+    for kind, i in (("window", 0), ("whole", 2)):
+        L = model._layers[i]
+        need = lib.rotor_b200_decoder_layer_workspace_bytes(C.byref(one), C.byref(L))
+        ws = torch.zeros(need, dtype=torch.uint8, device="cuda")
+        cache = model.runs[i].k_cache
+        weights = 2 * (row * d + h * (cfg["dim"] + cfg["vdim"]) * rank + d * h * cfg["vdim"] +
+                       (h * qd * d if kind == "window" else cfg["q_rank"] * (d + h * qd) + h * d))
+        for name, b, t, past in ((f"mixer_{kind}_prompt", B, S, 0), (f"mixer_{kind}_token_batch_1", 1, 1, S), (f"mixer_{kind}_token_batch_{B}", B, 1, S)):
+            run = lambda k, s: abi.check(lib.rotor_b200_latent_mixer(C.byref(one), C.byref(L), x.data_ptr(), b, t, past, cache.data_ptr(), -1,
+                                                                      y.data_ptr(), ws.data_ptr(), need, s))
+            sec = time_graph(torch, run, 2)
+            seen = sum(min(past + i + 1, W if kind == "window" else past + i + 1) for i in range(t))
+            flops = b * t * weights + 2.0 * b * h * seen * (qd + cfg["vdim"])    # (2 per weight, 2 bytes per weight)
+            keys = min(past + t, W + t - 1 if kind == "window" else past + t)
+            record(name, sec, weights + b * (keys * row * 2 + t * d * 6), flops if t > 1 else
+                   b * t * weights + 2.0 * b * h * seen * (row + rank))
+    expert = 2 * 3 * ff * d
+    spaces = []     # (a workspace holds one layer's layout)
+    for L in model._layers:
+        need = lib.rotor_b200_decoder_layer_workspace_bytes(C.byref(one), C.byref(L))
+        spaces.append((L, torch.zeros(need, dtype=torch.uint8, device="cuda"), need))
+    for m in (1, B, B * S):
+        run = lambda k, s: abi.check(lib.rotor_b200_experts(C.byref(one), C.byref(spaces[k][0]), x.data_ptr(), m, y.data_ptr(),
+                                                            spaces[k][1].data_ptr(), spaces[k][2], s))
+        sec = time_graph(torch, run, 3)
+        used = n * (1 - (1 - top / n) ** m)      # experts some token uses, on average
+        record(f"experts_rows_{m}", sec, used * expert + m * d * 6, m * top * expert)
+    abi.device_status()
+    return {"miborax_sublayers": out}
+
+
+def run_miborax(args):
+    """--workload miborax: prefill and decode throughput of the Miborax design beside Likerax with the same width, heads,
+    head size and feed-forward channels per token (random weights)."""
+    shapes = {"16h": (dict(MIBORAX_16H), args.layers or 6, args.batch or 8), "40h": (dict(MIBORAX_40H), min(args.layers or 3, 6), args.batch or 2)}
+    run_designs(args, "Miborax prefill and decode tokens/s beside Likerax at equal size", shapes,
+                {"miborax": lambda cfg, kw: miborax_random(cfg, cfg["n_layers"], **kw),
+                 "likerax": lambda cfg, kw: likerax_random(cfg, cfg["n_layers"], args.chunk, **kw)},
+                lambda torch, abi, cfg, B, S: dict(miborax_sublayers(torch, abi, cfg, B, S),
+                                                   likerax_kernels=likerax_kernels(torch, abi, cfg, B, S, args.chunk)))
 
 
 def time_prefill(torch, abi, model, vocab, B, S, K, W):
@@ -1038,17 +1156,18 @@ def main():
     ap.add_argument("--impl", default="b200", choices=["b200", "reference"])
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--quick", action="store_true", help="headline sections only (no parity / FFN / prefill / XL records)")
-    ap.add_argument("--only", default="all", choices=["all", "decode", "gemv", "gemm", "2b", "xl"],
+    ap.add_argument("--only", default="all", choices=["all", "decode", "gemv", "gemm", "2b", "xl", "16h", "40h"],
                     help="profiling aid: run only the device-resident decode section, the GEMV section, or one "
-                         "prefill GEMM (--m tokens); --workload likerax: one shape")
+                         "prefill GEMM (--m tokens); --workload likerax / miborax: one shape")
     ap.add_argument("--m", type=int, default=16384, help="--only gemm: activation columns (tokens)")
-    ap.add_argument("--workload", default="decode_2b", choices=["decode_2b", "xl_tp", "prefill_2b", "ffn_block", "likerax"],
+    ap.add_argument("--workload", default="decode_2b", choices=["decode_2b", "xl_tp", "prefill_2b", "ffn_block", "likerax", "miborax"],
                     help="decode_2b: the headline line; xl_tp: the tensor-parallel XL shape (separate line)")
     ap.add_argument("--batch", type=int, default=0, help="prefill_2b: sequences (0 = 8); xl_tp: sequences (0 = 1)")
     ap.add_argument("--seq", type=int, default=0, help="prefill_2b: positions per sequence (0 = 2048)")
     ap.add_argument("--layers", type=int, default=0, help="xl_tp: override the layer count (0 = 80)")
-    ap.add_argument("--family", default="both", choices=["both", "likerax", "bitnet"], help="likerax: which model")
-    ap.add_argument("--phase", default="both", choices=["both", "prefill", "decode"], help="likerax: which phase")
+    ap.add_argument("--family", default="both", choices=["both", "likerax", "bitnet", "miborax"],
+                    help="likerax / miborax: which model")
+    ap.add_argument("--phase", default="both", choices=["both", "prefill", "decode"], help="likerax / miborax: which phase")
     ap.add_argument("--chunk", type=int, default=4096, help="likerax: chunk length of the attention mask (0 = none)")
     ap.add_argument("--graph", type=int, default=1, help="xl_tp: replay the step as a CUDA graph (1) or launch it (0)")
     args = ap.parse_args()
@@ -1077,6 +1196,9 @@ def main():
     elif args.workload == "likerax":
         if rank == 0:
             run_likerax(args)
+    elif args.workload == "miborax":
+        if rank == 0:
+            run_miborax(args)
     elif args.workload == "ffn_block":
         if rank == 0:
             run_ffn_block(args)

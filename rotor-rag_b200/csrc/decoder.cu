@@ -216,7 +216,8 @@ static void carve_decoder(Model& m, DecoderStack& d, const rotor_b200_decoder_la
         d.route.counts = cv.take<int>(w.experts);
         d.route.cursor = cv.take<int>(w.experts);
         d.route.tile_rows = c.f32 ? 64 : 128;
-        d.route.table = cv.take<int>(1 + 3 * (size_t)route_tiles((long long)(rows * w.top), (int)w.experts, d.route.tile_rows));
+        d.route.max_tiles = route_tiles((long long)(rows * w.top), (int)w.experts, d.route.tile_rows);
+        d.route.table = cv.take<int>(1 + 3 * (size_t)d.route.max_tiles);
     }
     d.hn = cv.take<float>(rows * d.ldh);
     d.row_map = cv.take<int>(rows);
@@ -763,11 +764,7 @@ int rotor_b200_dense_linear(const void* w, int n, int k, const void* x, int rows
         p.y = static_cast<float*>(y);
         p.ldy = dense_ld(n);
     }
-    static PerDevice<bool> once;
-    if (!once.here()) {
-        RB_TRY(configure_dense());
-        once.here() = true;
-    }
+    RB_TRY(configure_dense());
     cudaStream_t st = as_stream(stream);
     if (dense_gemv_supported(p, rows)) return launch_dense_gemv(p, rows, st);
     return f32 ? launch_dense_gemm_f32(p, rows, scratch, st) : launch_dense_gemm_t5(p, rows, st);

@@ -73,7 +73,7 @@ struct Routing {
     int* counts;                 // [experts] zeroed words
     int* cursor;                 // [experts]
     int* table;                  // tiles of `tile_rows` slots: count, then (expert, first slot, slots) per tile
-    int tile_rows;
+    int tile_rows, max_tiles;    // (what counts that were not zeroed could say is cut to the table's size)
 };
 inline int route_tiles(long long slots, int experts, int tile_rows) { return (int)(slots / tile_rows) + experts; }
 // chooses the experts of every row, and copies the rows x (16-byte pieces) into their slots of `permuted`

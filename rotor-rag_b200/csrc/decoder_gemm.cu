@@ -510,6 +510,12 @@ int launch_dense_gemm_f32(const DenseProduct& p, int rows, float* gate_up, cudaS
 }
 
 int configure_dense_gemv();
-int configure_dense() { return configure_dense_gemv(); }
+int configure_dense() {
+    static PerDevice<bool> once;
+    if (once.here()) return ROTOR_B200_OK;
+    const int rc = configure_dense_gemv();
+    once.here() = rc == ROTOR_B200_OK;
+    return rc;
+}
 
 }  // namespace rb

@@ -29,12 +29,12 @@ __global__ void __launch_bounds__(256) route_choose_kernel(const __grid_constant
 }
 
 // One CTA of EXPERTS_MAX threads: first slot of every expert, the tile table; counts are zeroed for the next call.
-__global__ void __launch_bounds__(EXPERTS_MAX) route_table_kernel(const __grid_constant__ Routing r) {
+__global__ void __launch_bounds__(EXPERTS_MAX) route_table_kernel(const __grid_constant__ Routing r, int pairs) {
     __shared__ int2 warp_sums[32];
     pdl_wait();
     pdl_trigger();
     const int e = threadIdx.x, lane = e & 31, warp = e >> 5;
-    const int n = e < r.experts ? r.counts[e] : 0, tiles = (n + r.tile_rows - 1) / r.tile_rows;
+    const int n = e < r.experts ? min(max(r.counts[e], 0), pairs) : 0, tiles = (n + r.tile_rows - 1) / r.tile_rows;
     int2 s = make_int2(n, tiles);  // inclusive sums
     auto scan = [&]() {
 #pragma unroll
@@ -64,14 +64,14 @@ __global__ void __launch_bounds__(EXPERTS_MAX) route_table_kernel(const __grid_c
     if (e < r.experts) {
         r.cursor[e] = first;
         r.counts[e] = 0;
-        for (int t = 0; t < tiles; ++t) {
+        for (int t = 0; t < tiles && tile + t < r.max_tiles && first + t * r.tile_rows < pairs; ++t) {
             int* out = r.table + 1 + 3 * (tile + t);
             out[0] = e;
             out[1] = first + t * r.tile_rows;
-            out[2] = min(r.tile_rows, n - t * r.tile_rows);
+            out[2] = min(min(r.tile_rows, n - t * r.tile_rows), pairs - out[1]);
         }
     }
-    if (e == 0) r.table[0] = warp_sums[31].y;
+    if (e == 0) r.table[0] = min(warp_sums[31].y, r.max_tiles);
 }
 
 // One warp per (row, choice): takes the expert's next slot and copies the row there.
@@ -82,7 +82,7 @@ __global__ void __launch_bounds__(256) route_scatter_kernel(const __grid_constan
     for (int i = blockIdx.x * per + (threadIdx.x >> 5); i < pairs; i += gridDim.x * per) {
         int slot = 0;
         if (lane == 0) {
-            slot = atomicAdd(&r.cursor[r.chosen[i]], 1);
+            slot = min(max(atomicAdd(&r.cursor[r.chosen[i]], 1), 0), pairs - 1);
             r.slot_of[i] = slot;
         }
         slot = __shfl_sync(0xffffffffu, slot, 0);
@@ -97,8 +97,9 @@ int launch_route(const Routing& r, int rows, const void* x, size_t row_bytes, vo
     RB_REQUIRE(r.experts >= 1 && r.experts <= EXPERTS_MAX && r.top >= 1 && r.top <= r.experts && r.top <= EXPERT_TOP_MAX);
     RB_REQUIRE(row_bytes % 16 == 0 && (long long)rows * r.top < 0x7fffffffLL);
     const int pairs = rows * r.top, most = 148 * 8;
+    RB_REQUIRE(r.max_tiles >= route_tiles(pairs, r.experts, r.tile_rows));
     int rc = launch_chained(route_choose_kernel, dim3((rows + 7) / 8 < most ? (rows + 7) / 8 : most), dim3(256), 0, st, 1, r, rows);
-    if (!rc) rc = launch_chained(route_table_kernel, dim3(1), dim3(EXPERTS_MAX), 0, st, 1, r);
+    if (!rc) rc = launch_chained(route_table_kernel, dim3(1), dim3(EXPERTS_MAX), 0, st, 1, r, pairs);
     if (!rc)
         rc = launch_chained(route_scatter_kernel, dim3((pairs + 7) / 8 < most ? (pairs + 7) / 8 : most), dim3(256), 0, st, 1, r, pairs,
                             static_cast<const uint4*>(x), (int)(row_bytes / 16), static_cast<uint4*>(permuted));
