@@ -513,9 +513,10 @@ struct DecoderPass {
 
     int experts_ff(const rotor_b200_decoder_layer& L, const void* h, float* y, StreamStage* next) {
         const int lde = dense_ld(L.experts), ldf = dense_ld(L.ff);
+        Routing rt = d.route;
+        rt.early = routed;  // (by the input product: the mixer's launches lie between)
         if (!routed) RB_TRY(run(plain(L.router, L.experts, d.cfg.width, h, d.ld, d.logits, lde)));
         routed = false;
-        Routing rt = d.route;
         rt.logits = d.logits;
         rt.bias = L.router_b;
         rt.ld = lde;

@@ -66,6 +66,7 @@ struct Routing {
     const float* logits;         // [rows][ld]
     const float* bias;           // [experts], added to them; or null
     int ld, experts, top;
+    int early;                   // the outputs were written two or more launches ago: they may be read before the launch wait
     // many rows: filled by launch_route
     int* slot_of;                // [rows][top] slot of a token's k-th choice; slots of one expert are consecutive
     float* weight;               // [rows][top] softmax over the chosen logits
@@ -360,7 +361,8 @@ __device__ __forceinline__ void route_row(const Routing& r, int row, int lane, i
 template <int S>
 struct StreamGroup {
     float4 y, x[S ? S : 1];  // (a first stage keeps the embedding's columns in y)
-    __device__ __forceinline__ void load(const StreamStage& p, int row, int g) {
+    // slot, slot_w: the row's part of slot_of and slot_w, wherever it lies
+    __device__ __forceinline__ void load(const StreamStage& p, int row, int g, const int* slot, const float* slot_w) {
         if (p.ids) {
             long long id = p.ids[row];
             if (id < 0 || id >= p.vocab) id = 0;
@@ -376,13 +378,20 @@ struct StreamGroup {
             y.w += w * v.w;
         };
         if (p.y2) add(__ldcg(reinterpret_cast<const float4*>(p.y2 + (size_t)row * p.ld) + g), 1.f);
-        if (p.slots) {
-            for (int k = 0; k < p.top; ++k) {
-                const size_t at = (size_t)__ldcg(p.slot_of + (size_t)row * p.top + k) * p.ld;
-                const float w = __ldcg(p.slot_w + (size_t)row * p.top + k);
-                add(p.slots_f32 ? __ldcg(reinterpret_cast<const float4*>(static_cast<const float*>(p.slots) + at) + g)
-                                : bf16x4_to_float4(__ldcg(reinterpret_cast<const uint2*>(static_cast<const __nv_bfloat16*>(p.slots) + at) + g)),
-                    w);
+        if (p.slots && p.slots_f32) {
+            for (int k = 0; k < p.top; ++k)
+                add(__ldcg(reinterpret_cast<const float4*>(static_cast<const float*>(p.slots) + (size_t)slot[k] * p.ld) + g), slot_w[k]);
+        } else if (p.slots) {
+            constexpr int U = 4;  // slots requested together
+            for (int k0 = 0; k0 < p.top; k0 += U) {
+                uint2 v[U];
+#pragma unroll
+                for (int u = 0; u < U; ++u)
+                    if (k0 + u < p.top)
+                        v[u] = __ldcg(reinterpret_cast<const uint2*>(static_cast<const __nv_bfloat16*>(p.slots) + (size_t)slot[k0 + u] * p.ld) + g);
+#pragma unroll
+                for (int u = 0; u < U; ++u)
+                    if (k0 + u < p.top) add(bf16x4_to_float4(v[u]), slot_w[k0 + u]);
             }
         }
         if constexpr (S > 0) {

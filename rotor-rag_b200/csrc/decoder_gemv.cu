@@ -68,9 +68,13 @@ __global__ void __launch_bounds__(DG_THREADS, R <= 2 ? 2 : 1) dense_gemv_kernel(
         if constexpr (MODE == GV_EXPERT_DOWN) at += (size_t)s_sel[seg] * p.n;
         return w + at * p.ldw + lane * 8;
     };
-    if constexpr (EXPERT) {  // the weights depend on the router's outputs
-        pdl_wait();
-        pdl_trigger();
+    // the weights depend on the router's outputs; a down product's are older than the gated product in front of it
+    const bool late = MODE == GV_EXPERT_UP && !a.route.early;
+    if constexpr (EXPERT) {
+        if (late) {
+            pdl_wait();
+            pdl_trigger();
+        }
         const int row = MODE == GV_EXPERT_UP ? y / a.route.top : y;
         if (warp == 0) {
             int sel;
@@ -126,7 +130,7 @@ __global__ void __launch_bounds__(DG_THREADS, R <= 2 ? 2 : 1) dense_gemv_kernel(
             nw[i] = g < (a.st.ld >> 2) ? __ldg(reinterpret_cast<const float4*>(a.st.norm) + g) : make_float4(0.f, 0.f, 0.f, 0.f);
         }
     }
-    if constexpr (!EXPERT) {
+    if (!late) {
         pdl_wait();
         pdl_trigger();
     }
@@ -142,7 +146,7 @@ __global__ void __launch_bounds__(DG_THREADS, R <= 2 ? 2 : 1) dense_gemv_kernel(
                 StreamGroup<S> sg[SG];
 #pragma unroll
                 for (int i = 0; i < SG; ++i)
-                    if (g0 + i * DG_THREADS < n4) sg[i].load(s, r, g0 + i * DG_THREADS);
+                    if (g0 + i * DG_THREADS < n4) sg[i].load(s, r, g0 + i * DG_THREADS, s.slot_of + (size_t)r * s.top, s.slot_w + (size_t)r * s.top);
 #pragma unroll
                 for (int i = 0; i < SG; ++i) {
                     const int g = g0 + i * DG_THREADS;

@@ -9,7 +9,8 @@ namespace rb {
 template <int S>
 __global__ void __launch_bounds__(256) stream_stage_kernel(const __grid_constant__ StreamStage p, int rows) {
     extern __shared__ __align__(16) float us[];  // [ld]
-    __shared__ float coef[STREAMS_MAX * STREAMS_MAX + 2 * STREAMS_MAX], red[64];
+    __shared__ float coef[STREAMS_MAX * STREAMS_MAX + 2 * STREAMS_MAX], red[64], slot_w[EXPERT_TOP_MAX];
+    __shared__ int slot[EXPERT_TOP_MAX];
     stream_coefs(p, coef);
     pdl_wait();
     pdl_trigger();
@@ -18,13 +19,29 @@ __global__ void __launch_bounds__(256) stream_stage_kernel(const __grid_constant
     int k = 0;
     for (int r = blockIdx.x; r < rows; r += gridDim.x) {
         const int src = p.row_map ? p.row_map[r] : r;
+        if (p.slots) {
+            __syncthreads();  // (the row before is done with them)
+            if ((int)threadIdx.x < p.top) {
+                slot[threadIdx.x] = __ldcg(p.slot_of + (size_t)src * p.top + threadIdx.x);
+                slot_w[threadIdx.x] = __ldcg(p.slot_w + (size_t)src * p.top + threadIdx.x);
+            }
+            __syncthreads();
+        }
         float ss = 0.f;
-        for (int g = threadIdx.x; g < n4; g += blockDim.x) {
-            StreamGroup<S> sg;
-            sg.load(p, src, g);
-            const float4 u = sg.finish(p, coef, src, g, p.x_out != nullptr);
-            ss += p.norm_b ? u.x + u.y + u.z + u.w : u.x * u.x + u.y * u.y + u.z * u.z + u.w * u.w;
-            reinterpret_cast<float4*>(us)[g] = u;
+        constexpr int U = S == 1 ? 2 : 1;  // groups per thread requested together
+        for (int g0 = threadIdx.x; g0 < n4; g0 += U * blockDim.x) {
+            StreamGroup<S> sg[U];
+#pragma unroll
+            for (int i = 0; i < U; ++i)
+                if (g0 + i * (int)blockDim.x < n4) sg[i].load(p, src, g0 + i * blockDim.x, slot, slot_w);
+#pragma unroll
+            for (int i = 0; i < U; ++i) {
+                const int g = g0 + i * blockDim.x;
+                if (g >= n4) break;
+                const float4 u = sg[i].finish(p, coef, src, g, p.x_out != nullptr);
+                ss += p.norm_b ? u.x + u.y + u.z + u.w : u.x * u.x + u.y * u.y + u.z * u.z + u.w * u.w;
+                reinterpret_cast<float4*>(us)[g] = u;
+            }
         }
         if (!p.h) continue;
         float mean = 0.f;

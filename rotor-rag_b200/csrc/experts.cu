@@ -74,21 +74,35 @@ __global__ void __launch_bounds__(EXPERTS_MAX) route_table_kernel(const __grid_c
     if (e == 0) r.table[0] = min(warp_sums[31].y, r.max_tiles);
 }
 
-// One warp per (row, choice): takes the expert's next slot and copies the row there.
-__global__ void __launch_bounds__(256) route_scatter_kernel(const __grid_constant__ Routing r, int pairs, const uint4* x, int pieces, uint4* permuted) {
+// One warp per row: takes the next slot of each of its experts and copies the row there, read once.
+__global__ void __launch_bounds__(256) route_scatter_kernel(const __grid_constant__ Routing r, int rows, const uint4* x, int pieces, uint4* permuted) {
     pdl_wait();
     pdl_trigger();
-    const int lane = threadIdx.x & 31, per = blockDim.x >> 5;
-    for (int i = blockIdx.x * per + (threadIdx.x >> 5); i < pairs; i += gridDim.x * per) {
+    const int lane = threadIdx.x & 31, per = blockDim.x >> 5, pairs = rows * r.top;
+    constexpr int U = 4;  // pieces per lane requested together
+    for (int row = blockIdx.x * per + (threadIdx.x >> 5); row < rows; row += gridDim.x * per) {
+        const uint4* src = x + (size_t)row * pieces;
+        uint4 v[U];
+        auto fetch = [&](int c0) {
+#pragma unroll
+            for (int u = 0; u < U; ++u)
+                if (c0 + 32 * u + lane < pieces) v[u] = __ldg(src + c0 + 32 * u + lane);
+        };
+        fetch(0);
         int slot = 0;
-        if (lane == 0) {
-            slot = min(max(atomicAdd(&r.cursor[r.chosen[i]], 1), 0), pairs - 1);
-            r.slot_of[i] = slot;
+        if (lane < r.top) {
+            slot = min(max(atomicAdd(&r.cursor[r.chosen[(size_t)row * r.top + lane]], 1), 0), pairs - 1);
+            r.slot_of[(size_t)row * r.top + lane] = slot;
         }
-        slot = __shfl_sync(0xffffffffu, slot, 0);
-        const uint4* src = x + (size_t)(i / r.top) * pieces;
-        uint4* dst = permuted + (size_t)slot * pieces;
-        for (int c = lane; c < pieces; c += 32) dst[c] = __ldg(src + c);
+        for (int c0 = 0; c0 < pieces; c0 += 32 * U) {
+            if (c0) fetch(c0);
+            for (int k = 0; k < r.top; ++k) {
+                uint4* dst = permuted + (size_t)__shfl_sync(0xffffffffu, slot, k) * pieces;
+#pragma unroll
+                for (int u = 0; u < U; ++u)
+                    if (c0 + 32 * u + lane < pieces) dst[c0 + 32 * u + lane] = v[u];
+            }
+        }
     }
 }
 
@@ -101,7 +115,7 @@ int launch_route(const Routing& r, int rows, const void* x, size_t row_bytes, vo
     int rc = launch_chained(route_choose_kernel, dim3((rows + 7) / 8 < most ? (rows + 7) / 8 : most), dim3(256), 0, st, 1, r, rows);
     if (!rc) rc = launch_chained(route_table_kernel, dim3(1), dim3(EXPERTS_MAX), 0, st, 1, r, pairs);
     if (!rc)
-        rc = launch_chained(route_scatter_kernel, dim3((pairs + 7) / 8 < most ? (pairs + 7) / 8 : most), dim3(256), 0, st, 1, r, pairs,
+        rc = launch_chained(route_scatter_kernel, dim3((rows + 7) / 8 < most ? (rows + 7) / 8 : most), dim3(256), 0, st, 1, r, rows,
                             static_cast<const uint4*>(x), (int)(row_bytes / 16), static_cast<uint4*>(permuted));
     return rc;
 }

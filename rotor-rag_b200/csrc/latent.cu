@@ -9,8 +9,8 @@
 // the row's visible positions for one tile of heads, walks it in tiles of cache rows staged by cp.async (the
 // first requested before the programmatic-launch wait where it holds only rows of earlier steps), keeps a
 // running maximum and sum per head, and the cluster merges through distributed shared memory.
-//   bf16:    16 heads a tile are the M of mma.m16n8k16: warps split the positions for the scores and the
-//            latent columns for the sums
+//   bf16:    16 heads a tile are the M of mma.m16n8k16: warps split the positions and halves of a row for the
+//            scores and the latent columns for the sums
 //   float32: the FP32 pipe, eight heads a tile
 #include <type_traits>
 
@@ -18,9 +18,9 @@
 
 namespace rb {
 
-constexpr int LA_THREADS = 256, LA_WARPS = LA_THREADS / 32;
+constexpr int LA_THREADS = 512, LA_WARPS = LA_THREADS / 32;
 constexpr int LA_HEADS = 16, LF_HEADS = 8;
-constexpr int LA_MAX_SPLITS = 8;
+constexpr int LA_MAX_SPLITS = 16;           // (above eight: clusters of a size the device has to allow)
 constexpr size_t LA_SMEM_MAX = 200 * 1024;
 
 struct LatentArgs {
@@ -98,23 +98,42 @@ int launch_latent_finish(const LatentFinish& p, int rows, cudaStream_t st) {
                  : launch_chained(latent_finish_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, 1, p, rows);
 }
 
+// One CTA per row.
 template <typename T>
 __global__ void __launch_bounds__(256) rms_rows_kernel(const float* x, int ldx, int n, const float* norm, float eps, T* out, int ldo, int rows) {
+    __shared__ float red[64];
     pdl_wait();
     pdl_trigger();
-    const int lane = threadIdx.x & 31, per = blockDim.x >> 5;
-    for (int r = blockIdx.x * per + (threadIdx.x >> 5); r < rows; r += gridDim.x * per) {
-        const float* v = x + (size_t)r * ldx;
+    int k = 0;
+    for (int r = blockIdx.x; r < rows; r += gridDim.x) {
+        const float2* v = reinterpret_cast<const float2*>(x + (size_t)r * ldx);
+        constexpr int U = 4;  // column pairs per thread that stay in registers
+        float2 keep[U];
         float ss = 0.f;
-        for (int c = lane; c < n; c += 32) ss += v[c] * v[c];
-        const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)n + eps);
-        for (int c = lane; c < ldo; c += 32) la_store(out + (size_t)r * ldo + c, c < n ? v[c] * inv * __ldg(norm + c) : 0.f);
+        auto pair = [&](int c) {
+            float2 q = 2 * c < n ? v[c] : make_float2(0.f, 0.f);
+            if (2 * c + 1 >= n) q.y = 0.f;
+            ss += q.x * q.x + q.y * q.y;
+            return q;
+        };
+#pragma unroll
+        for (int u = 0; u < U; ++u) keep[u] = pair(threadIdx.x + u * blockDim.x);
+        for (int c = threadIdx.x + U * blockDim.x; 2 * c < n; c += blockDim.x) pair(c);
+        const float inv = 1.0f / sqrtf(block_sum_alt(ss, red, k) / (float)n + eps);
+        auto put = [&](int c, const float2 q) {
+            if (2 * c < ldo)
+                la_store2(out + (size_t)r * ldo + 2 * c, make_float2(2 * c < n ? q.x * inv * __ldg(norm + 2 * c) : 0.f,
+                                                                     2 * c + 1 < n ? q.y * inv * __ldg(norm + 2 * c + 1) : 0.f));
+        };
+#pragma unroll
+        for (int u = 0; u < U; ++u) put(threadIdx.x + u * blockDim.x, keep[u]);
+        for (int c = threadIdx.x + U * blockDim.x; 2 * c < ldo; c += blockDim.x) put(c, pair(c));
     }
 }
 
 int launch_rms_rows(const float* x, int ldx, int n, const float* norm, float eps, void* out, int ldo, int f32, int rows, cudaStream_t st) {
-    RB_REQUIRE(x && norm && out && rows > 0 && n > 0 && n <= ldo);
-    const dim3 grid((rows + 7) / 8 < 148 * 8 ? (rows + 7) / 8 : 148 * 8);
+    RB_REQUIRE(x && norm && out && rows > 0 && n > 0 && n <= ldo && ldx % 2 == 0 && ldo % 2 == 0);
+    const dim3 grid(rows < 148 * 8 ? rows : 148 * 8);
     return f32 ? launch_chained(rms_rows_kernel<float>, grid, dim3(256), 0, st, 1, x, ldx, n, norm, eps, static_cast<float*>(out), ldo, rows)
                : launch_chained(rms_rows_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, 1, x, ldx, n, norm, eps,
                                 static_cast<__nv_bfloat16*>(out), ldo, rows);
@@ -154,13 +173,13 @@ struct LatentRun {
     // cache rows k0 .. k0 + tile - 1 below t1, `skip` left out; rows behind them as zeros
     __device__ __forceinline__ void load(T* dst, int k0, int tile, int skip) const {
         const int n = min(tile, t1 - k0), pieces = W / PIECE;
-        for (int i = threadIdx.x; i < tile * pieces; i += LA_THREADS) {
-            const int j = i / pieces, c = i - j * pieces;
+        for (int j = threadIdx.x >> 5; j < tile; j += LA_WARPS) {
             if (k0 + j == skip && j < n) continue;
             const int bytes = j < n ? 16 : 0;
-            const T* src = rows + (size_t)(j < n ? k0 + j : k0) * W + c * PIECE;
-            asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(la_smem(dst + (size_t)j * stride + c * PIECE)), "l"(src), "r"(bytes)
-                         : "memory");
+            const T* src = rows + (size_t)(j < n ? k0 + j : k0) * W;
+            const uint32_t to = la_smem(dst + (size_t)j * stride);
+            for (int c = threadIdx.x & 31; c < pieces; c += 32)
+                asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(to + 16 * c), "l"(src + c * PIECE), "r"(bytes) : "memory");
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     }
@@ -263,8 +282,8 @@ __global__ void __launch_bounds__(LA_THREADS) latent_attn_mma_kernel(const __gri
     T* qs = reinterpret_cast<T*>(la_raw);                        // [16][ws]
     T* kv = qs + LA_HEADS * ws;                                  // [2][TK][ws]; at the end the CTA's sums, float [16][kp + 4]
     T* ps = kv + 2 * (size_t)TK * ws;                            // [16][TK + 8] weights
-    float* sc = reinterpret_cast<float*>(ps + LA_HEADS * ps_ld); // [16][TK + 4] scores
-    float* ml = sc + LA_HEADS * ss;                              // m [16], l [16], alpha [16]
+    float* sc = reinterpret_cast<float*>(ps + LA_HEADS * ps_ld); // [2][16][TK + 4] scores, by halves of the row
+    float* ml = sc + 2 * LA_HEADS * ss;                             // m [16], l [16], alpha [16]
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const float2* rope = p.cache.rope + (size_t)run.pos * (s.rot >> 1);
     const int skip = p.dkv ? run.pos : -1;
@@ -311,42 +330,53 @@ __global__ void __launch_bounds__(LA_THREADS) latent_attn_mma_kernel(const __gri
             asm volatile("cp.async.wait_group 0;" ::: "memory");
         }
         __syncthreads();
-        // scores of eight positions per warp
-        for (int kb = warp * 8; kb < TK; kb += LA_WARPS * 8) {
-            float d0[4] = {0.f, 0.f, 0.f, 0.f}, d1[4] = {0.f, 0.f, 0.f, 0.f};
-            const uint32_t ka = la_smem(tile + (size_t)(kb + (lane & 7)) * ws + (lane >> 3) * 8);
-            int c = 0;
-            for (; c + 32 <= W; c += 32) {
-                uint32_t q0[4], q1[4], b[4];
-                la_ldm4(b, ka + c * 2);
-                la_ldm4(q0, qa + c * 2);
-                la_ldm4(q1, qa + c * 2 + 32);
-                la_mma(d0, q0, b[0], b[1]);
-                la_mma(d1, q1, b[2], b[3]);
+        // scores of eight positions per warp, over half of the row
+        {
+            const int kb = (warp & 7) * 8, part = warp >> 3, mid = (W / 16 + 1) / 2 * 16;
+            if (kb < TK) {
+                float d0[4] = {0.f, 0.f, 0.f, 0.f}, d1[4] = {0.f, 0.f, 0.f, 0.f};
+                const uint32_t ka = la_smem(tile + (size_t)(kb + (lane & 7)) * ws + (lane >> 3) * 8);
+                const int end = part ? W : mid;
+                int c = part ? mid : 0;
+#pragma unroll 3
+                for (; c + 32 <= end; c += 32) {
+                    uint32_t q0[4], q1[4], b[4];
+                    la_ldm4(b, ka + c * 2);
+                    la_ldm4(q0, qa + c * 2);
+                    la_ldm4(q1, qa + c * 2 + 32);
+                    la_mma(d0, q0, b[0], b[1]);
+                    la_mma(d1, q1, b[2], b[3]);
+                }
+                if (c < end) {
+                    uint32_t q0[4], b0, b1;
+                    const uint32_t kt = la_smem(tile + (size_t)(kb + (lane & 7)) * ws + ((lane >> 3) & 1) * 8 + c);
+                    asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0, %1}, [%2];" : "=r"(b0), "=r"(b1) : "r"(kt));
+                    la_ldm4(q0, qa + c * 2);
+                    la_mma(d0, q0, b0, b1);
+                }
+                float* to = sc + (size_t)part * LA_HEADS * ss + (lane >> 2) * ss + kb + (lane & 3) * 2;
+                *reinterpret_cast<float2*>(to) = make_float2(d0[0] + d1[0], d0[1] + d1[1]);
+                *reinterpret_cast<float2*>(to + 8 * ss) = make_float2(d0[2] + d1[2], d0[3] + d1[3]);
             }
-            if (c < W) {
-                uint32_t q0[4], b0, b1;
-                const uint32_t kt = la_smem(tile + (size_t)(kb + (lane & 7)) * ws + ((lane >> 3) & 1) * 8 + c);
-                asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0, %1}, [%2];" : "=r"(b0), "=r"(b1) : "r"(kt));
-                la_ldm4(q0, qa + c * 2);
-                la_mma(d0, q0, b0, b1);
-            }
-            const int r = lane >> 2, k = kb + (lane & 3) * 2;
-#pragma unroll
-            for (int e = 0; e < 4; ++e)
-                sc[(r + (e >> 1) * 8) * ss + k + (e & 1)] = k + (e & 1) < n ? (d0[e] + d1[e]) * scale2 : -INFINITY;
         }
         __syncthreads();
+        static_assert(LA_HEADS == LA_WARPS, "a warp per head");
+        {
+            const int h = warp;
+            float v[2], top = -INFINITY, sum = 0.f;  // (tiles of up to 64 positions)
 #pragma unroll
-        for (int q = 0; q < LA_HEADS / LA_WARPS; ++q) {
-            const int h = warp + q * LA_WARPS;
-            float top = -INFINITY, sum = 0.f;
-            for (int k = lane; k < TK; k += 32) top = fmaxf(top, sc[h * ss + k]);
+            for (int i = 0; i < 2; ++i) {
+                const int k = lane + 32 * i;
+                v[i] = k < n ? (sc[h * ss + k] + sc[(LA_HEADS + h) * ss + k]) * scale2 : -INFINITY;
+                top = fmaxf(top, v[i]);
+            }
             const float m_old = ml[h], m_new = fmaxf(m_old, warp_max(top));  // finite: a tile has a visible position
-            for (int k = lane; k < TK; k += 32) {
-                const float e = exp2f(sc[h * ss + k] - m_new);
-                ps[h * ps_ld + k] = __float2bfloat16_rn(e);
-                sum += e;
+#pragma unroll
+            for (int i = 0; i < 2; ++i) {
+                const int k = lane + 32 * i;
+                v[i] = exp2f(v[i] - m_new);
+                if (k < TK) ps[h * ps_ld + k] = __float2bfloat16_rn(v[i]);
+                sum += v[i];
             }
             sum = warp_sum(sum);
             if (lane == 0) {
@@ -493,7 +523,7 @@ static size_t la_bytes(const LatentShape& s, int f32, int tile) {
     size_t kv = 2 * (size_t)tile * (W + 8) * 2;
     const size_t sums = (size_t)LA_HEADS * (s.kp + 4) * sizeof(float);
     if (kv < sums) return 0;
-    return LA_HEADS * (W + 8) * 2 + kv + LA_HEADS * (size_t)(tile + 8) * 2 + LA_HEADS * (size_t)(tile + 4) * sizeof(float) + 3 * LA_HEADS * sizeof(float);
+    return LA_HEADS * (W + 8) * 2 + kv + LA_HEADS * (size_t)(tile + 8) * 2 + 2 * LA_HEADS * (size_t)(tile + 4) * sizeof(float) + 3 * LA_HEADS * sizeof(float);
 }
 static int la_tile(const LatentShape& s, int f32) {
     for (int tile = 64; tile >= (f32 ? 8 : 16); tile >>= 1) {
@@ -506,20 +536,49 @@ bool latent_attn_supported(const LatentShape& s, int f32) {
     return s.heads > 0 && s.kp > 0 && s.rp >= 0 && s.kp % 16 == 0 && s.rp % 16 == 0 && (f32 || s.kp <= 1024) && la_tile(s, f32) > 0;
 }
 
-static int la_configure() {
-    static PerDevice<bool> once;
-    if (once.here()) return ROTOR_B200_OK;
-    void (*const kernels[])(LatentArgs) = {latent_attn_f32_kernel, latent_attn_mma_kernel<1>, latent_attn_mma_kernel<2>, latent_attn_mma_kernel<4>,
-                                           latent_attn_mma_kernel<8>};
-    for (auto k : kernels) RB_CUDA(cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)LA_SMEM_MAX));
-    once.here() = true;
-    return ROTOR_B200_OK;
+typedef void (*LatentKernel)(LatentArgs);
+static LatentKernel la_kernel(const LatentShape& s, int f32) {
+    if (f32) return latent_attn_f32_kernel;
+    return s.kp <= 256 ? latent_attn_mma_kernel<1> : s.kp <= 512 ? latent_attn_mma_kernel<2> : latent_attn_mma_kernel<4>;
 }
 
-static int la_go(void (*kernel)(LatentArgs), const LatentArgs& a, int rows, int splits, int head_tiles, size_t smem, cudaStream_t st) {
-    const int rc = la_configure();
-    if (rc) return rc;
-    return launch_chained(kernel, dim3(splits, head_tiles, rows), dim3(LA_THREADS), smem, st, splits, a);
+// Sets the kernels up; whether the device places clusters of sixteen of this one.
+static int la_configure(LatentKernel kernel, size_t smem, bool* sixteen) {
+    static PerDevice<bool> once;
+    if (!once.here()) {
+        for (LatentKernel k : {(LatentKernel)latent_attn_f32_kernel, (LatentKernel)latent_attn_mma_kernel<1>, (LatentKernel)latent_attn_mma_kernel<2>,
+                               (LatentKernel)latent_attn_mma_kernel<4>}) {
+            RB_CUDA(cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)LA_SMEM_MAX));
+            RB_CUDA(cudaFuncSetAttribute(k, cudaFuncAttributeNonPortableClusterSizeAllowed, 1));
+        }
+        once.here() = true;
+    }
+    struct Known {
+        LatentKernel kernel;
+        size_t smem;
+        bool sixteen;
+    };
+    static PerDevice<Known> last;
+    Known& known = last.here();
+    if (known.kernel != kernel || known.smem != smem) {
+        cudaLaunchConfig_t cfg = {};
+        cfg.gridDim = dim3(LA_MAX_SPLITS);
+        cfg.blockDim = dim3(LA_THREADS);
+        cfg.dynamicSmemBytes = smem;
+        cudaLaunchAttribute attr[1];
+        attr[0].id = cudaLaunchAttributeClusterDimension;
+        attr[0].val.clusterDim.x = LA_MAX_SPLITS;
+        attr[0].val.clusterDim.y = 1;
+        attr[0].val.clusterDim.z = 1;
+        cfg.attrs = attr;
+        cfg.numAttrs = 1;
+        int clusters = 0;
+        const bool ok = cudaOccupancyMaxActiveClusters(&clusters, kernel, &cfg) == cudaSuccess && clusters > 0;
+        cudaGetLastError();
+        known = {kernel, smem, ok};
+    }
+    *sixteen = known.sixteen;
+    return ROTOR_B200_OK;
 }
 
 int launch_latent_attn(const LatentAttn& p, int rows, cudaStream_t st) {
@@ -532,18 +591,19 @@ int launch_latent_attn(const LatentAttn& p, int rows, cudaStream_t st) {
     a.p = p;
     a.tile = la_tile(p.s, p.f32);
     const size_t smem = la_bytes(p.s, p.f32, a.tile);
+    const LatentKernel kernel = la_kernel(p.s, p.f32);
+    bool sixteen;
+    const int rc = la_configure(kernel, smem, &sixteen);
+    if (rc) return rc;
     for (int r0 = 0; r0 < rows; r0 += 65535) {  // (the grid's z limit)
         const int n = rows - r0 < 65535 ? rows - r0 : 65535;
+        const long long ctas = (long long)n * head_tiles;
         int splits = 1;
-        while (splits < LA_MAX_SPLITS && (long long)n * head_tiles * splits * 2 <= 148 && reach >= 32 * splits) splits *= 2;
+        while (splits < 8 && ctas * splits * 2 <= 148 && reach >= 32 * splits) splits *= 2;
+        if (splits == 8 && sixteen && ctas <= 4 && reach >= 512) splits = 16;  // (a cluster of sixteen fills most of a GPC)
         a.row0 = r0;
-        int rc;
-        if (p.f32) rc = la_go(latent_attn_f32_kernel, a, n, splits, head_tiles, smem, st);
-        else if (p.s.kp <= 128) rc = la_go(latent_attn_mma_kernel<1>, a, n, splits, head_tiles, smem, st);
-        else if (p.s.kp <= 256) rc = la_go(latent_attn_mma_kernel<2>, a, n, splits, head_tiles, smem, st);
-        else if (p.s.kp <= 512) rc = la_go(latent_attn_mma_kernel<4>, a, n, splits, head_tiles, smem, st);
-        else rc = la_go(latent_attn_mma_kernel<8>, a, n, splits, head_tiles, smem, st);
-        if (rc) return rc;
+        const int e = launch_chained(kernel, dim3(splits, head_tiles, n), dim3(LA_THREADS), smem, st, splits, a);
+        if (e) return e;
     }
     return ROTOR_B200_OK;
 }
