@@ -10,7 +10,7 @@
 //   up to DENSE_FEW_ROWS rows: the stages ride in the input products' prologues
 // Mixers, many rows / generation step
 //   bias:    [head finish ->] attention              / attention (normalises and appends its own row)
-//   latent:  [query latent norm, product ->] finish -> expansion of the cached latents -> attention (prompts), or
+//   latent:  [query latent norm, product (rotates) ->] finish -> expansion of the cached latents -> attention (prompts), or
 //            finish -> absorbing product -> attention -> value product
 //                                                    / [product ->] absorbing product -> attention (rotates,
 //                                                      norms and appends its own row) -> value product
@@ -380,7 +380,27 @@ struct DecoderPass {
         first.n = cols.all;
         first.y = d.qkv;
         first.ldy = ld_in;
-        RB_TRY(staged ? run_staged(first) : run(first));
+        const bool expanded = !f32 && expanded_attn_supported(s, seq) && expand != 0;
+        // prompts: the queries are rotated in the read-back of the product that makes them, where the head sizes allow
+        auto turning = [&](DenseProduct p) {
+            p.epilogue = DENSE_ROPE;
+            p.q_cols = s.heads * qd;
+            p.rot_at = s.dp;
+            p.rot = s.rot == s.rp ? s.rot : 0;
+            p.rope = reinterpret_cast<const float2*>(L.rope);
+            p.cache = {nullptr, nullptr, m.c.d_pos, d.cfg.max_seq, seq};
+            p.q = static_cast<__nv_bfloat16*>(d.lq);
+            p.n2 = 0;
+            return p;
+        };
+        bool turned = false;
+        if (expanded && !few && !m.no_fused && !L.q_rank && dense_gemm_t5_supported(turning(first), rows)) {
+            turned = true;
+            if (staged) RB_TRY(launch_stream_stage(sg, rows, st));
+            RB_TRY(many(turning(first), rows));
+        } else {
+            RB_TRY(staged ? run_staged(first) : run(first));
+        }
         const float* dkv = L.own_kv ? d.qkv + cols.q : nullptr;
         const float* gate = L.gated ? d.qkv + cols.q + cols.dkv : nullptr;
         const float* q = d.qkv;
@@ -396,7 +416,9 @@ struct DecoderPass {
             } else {
                 const int ldc = dense_ld(L.q_rank);
                 RB_TRY(launch_rms_rows(d.qkv, ld_in, L.q_rank, L.q_norm, d.cfg.eps, d.cq, ldc, f32, rows, st));
-                RB_TRY(many(plain(L.uq, s.heads * qd, L.q_rank, d.cq, ldc, d.q_raw, ldq), rows));
+                const DenseProduct uq = plain(L.uq, s.heads * qd, L.q_rank, d.cq, ldc, d.q_raw, ldq);
+                turned = expanded && !m.no_fused && dense_gemm_t5_supported(turning(uq), rows);
+                RB_TRY(many(turned ? turning(uq) : uq, rows));
             }
             q = d.q_raw;
         }
@@ -410,8 +432,8 @@ struct DecoderPass {
         fin.ld_dkv = ld_in;
         fin.dkv_norm = L.kv_norm;
         fin.q_out = d.lq;
-        if (!f32 && expanded_attn_supported(s, seq) && expand != 0) {
-            fin.q = q;
+        if (expanded) {
+            fin.q = turned ? nullptr : q;
             RB_TRY(launch_latent_finish(fin, rows, st));
             const int first_pos = L.window > 0 && m.past - L.window + 1 > 0 ? m.past - L.window + 1 : 0, len = m.past + seq - first_pos;
             const int cols_kv = s.heads * (s.dp + vp), step = d.kv_rows / len;

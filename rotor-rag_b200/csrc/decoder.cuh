@@ -57,7 +57,7 @@ struct StreamStage {
 };
 int launch_stream_stage(const StreamStage& p, int rows, cudaStream_t st);
 
-enum DenseEpilogue { DENSE_PLAIN = 0, DENSE_GATED = 1, DENSE_QKV = 2, DENSE_HALF = 3 };
+enum DenseEpilogue { DENSE_PLAIN = 0, DENSE_GATED = 1, DENSE_QKV = 2, DENSE_HALF = 3, DENSE_ROPE = 4 };
 enum GateAct { ACT_GELU_TANH = 0, ACT_SILU = 1 };
 constexpr int EXPERTS_MAX = 1024, EXPERT_TOP_MAX = 32;
 
@@ -117,6 +117,10 @@ struct DenseProduct {
     HeadShape shape;
     CacheView cache;
     __nv_bfloat16* q;            // [rows][heads * kd]
+    // DENSE_ROPE (bf16): the first q_cols outputs are query heads of rot_at plain and rot columns to be rotated by their
+    // token's position, bf16 rows of their own in q; the rest is float32 in y
+    int q_cols, rot_at, rot;
+    const float2* rope;          // [max_seq][rot / 2]
     // groups (0 means 1): distances in elements (x columns and rows, w rows, output columns and rows)
     int groups, gx_col, gx_row, gw_row, gy_col, gy_row;
     const float* head_gate;

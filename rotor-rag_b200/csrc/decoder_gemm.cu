@@ -9,6 +9,8 @@
 //   PLAIN  float32
 //   HALF   bf16, optionally times the sigmoid of a gate per token and group
 //   GATED  a tile holds BN/2 gate rows and the matching up rows; act(gate) * up as bf16
+//   ROPE   query heads with their rotated columns turned by the token's position as bf16 rows, what lies behind
+//          them as float32
 //   QKV    the heads of the stacked q/k/v matrix: q and k divided by their root mean square, q rows
 //          out, k and v rows to the cache positions of their tokens
 // Groups (heads, sequences, experts) are more tiles of the same launch: a tile's operand and output origins
@@ -45,6 +47,8 @@ struct DgT5Params {
     int act, groups, gx_col, gx_row, gw_row, gy_col, gy_row;
     const float* head_gate;
     int ld_head_gate;
+    int q_cols, rot_at, rot;
+    const float2* rope;
     const int* table;             // experts: tile count, then (expert, first slot, slots) per tile of tokens
 };
 
@@ -215,6 +219,42 @@ dense_gemm_t5_kernel(const __grid_constant__ CUtensorMap tm_a, const __grid_cons
                         return tok0 + tl < tok_end && col + piece < p.n ? p.a + (size_t)(tok0 + tl) * p.lda + at.y_col + col : nullptr;
                     });
                 }
+            } else if constexpr (EPI == DENSE_ROPE) {
+                const int tok = min(tok0 + lane, p.rows - 1), b = tok / p.cache.seq;
+                const int pos = min(cached_len(p.cache.past_len, b, p.cache.max_seq) + (tok - b * p.cache.seq), p.cache.max_seq - 1);
+                const float2* rope = p.rope + (size_t)pos * (p.rot >> 1);
+                const int qd = p.rot_at + p.rot;
+#pragma unroll 1
+                for (int c = 0; c < BN / 32; ++c) {
+                    const int col = n * TN + c * 32;
+                    if (col >= p.ldy) break;
+                    uint32_t v[32];
+                    t5_ld32(tb + c * 32, v);
+                    asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+                    if (col >= p.q_cols) {
+                        t5_store_rows(stage, v, p.y + (size_t)tok0 * p.ldy + col, (size_t)p.ldy * 4, tok0, tok_end, lane);
+                        continue;
+                    }
+                    uint32_t o[16];
+                    const int turn = col % qd - p.rot_at;  // (columns of a chunk are all plain or all rotated)
+                    if (turn < 0) {
+#pragma unroll
+                        for (int i = 0; i < 16; ++i) o[i] = t5_pack(__uint_as_float(v[2 * i]), __uint_as_float(v[2 * i + 1]));
+                    } else {
+                        const float4* cs = reinterpret_cast<const float4*>(rope + (turn >> 1));
+#pragma unroll
+                        for (int i = 0; i < 8; ++i) {
+                            const float4 t = __ldg(cs + i);
+                            const float a = __uint_as_float(v[4 * i]), b2 = __uint_as_float(v[4 * i + 1]), e = __uint_as_float(v[4 * i + 2]),
+                                        f = __uint_as_float(v[4 * i + 3]);
+                            o[2 * i] = t5_pack(a * t.x - b2 * t.y, b2 * t.x + a * t.y);
+                            o[2 * i + 1] = t5_pack(e * t.z - f * t.w, f * t.z + e * t.w);
+                        }
+                    }
+                    t5_store_half_rows_to(stage, o, lane, [&](int tl) -> void* {
+                        return tok0 + tl < tok_end ? p.q + (size_t)(tok0 + tl) * p.q_cols + col : nullptr;
+                    });
+                }
             } else if constexpr (EPI == DENSE_GATED) {
 #pragma unroll 1
                 for (int c = 0; c < TN / 32; ++c) {
@@ -305,6 +345,8 @@ bool dense_gemm_t5_supported(const DenseProduct& p, int rows) {
     if (p.f32 || rows < 1 || p.ldw % 8 || p.ldx % 8 || ((uintptr_t)p.w & 15) || ((uintptr_t)p.x & 15)) return false;
     if (p.epilogue == DENSE_PLAIN) return p.ldy % 32 == 0;
     if (p.epilogue == DENSE_GATED) return p.lda % 32 == 0;
+    if (p.epilogue == DENSE_ROPE)
+        return p.ldy % 32 == 0 && p.rot_at % 32 == 0 && p.rot % 32 == 0 && p.rot > 0 && p.q_cols % (p.rot_at + p.rot) == 0 && !p.groups && !p.route;
     if (p.epilogue == DENSE_HALF) return p.lda % 8 == 0 && (!p.groups || p.n % 8 == 0) && p.gy_col % 8 == 0 && p.gx_col % 8 == 0;
     // heads that never straddle a 64-column tile, cache rows without padding
     const HeadShape& s = p.shape;
@@ -351,6 +393,10 @@ static int dg5_launch(const DenseProduct& p, int rows, cudaStream_t st) {
     a.gy_row = p.gy_row;
     a.head_gate = p.head_gate;
     a.ld_head_gate = p.ld_head_gate;
+    a.q_cols = p.q_cols;
+    a.rot_at = p.rot_at;
+    a.rot = p.rot;
+    a.rope = p.rope;
     a.table = p.route ? p.route->table : nullptr;
     // extents of the operands, all groups together
     const size_t x_rows = (size_t)rows + (size_t)(groups - 1) * p.gx_row, x_cols = (size_t)p.k + (size_t)(groups - 1) * p.gx_col;
@@ -379,6 +425,9 @@ int launch_dense_gemm_t5(const DenseProduct& p, int rows, cudaStream_t st) {
         case DENSE_HALF:
             if (wide) return dg5_launch<256, DENSE_HALF>(p, rows, st);
             return narrow ? dg5_launch<32, DENSE_HALF>(p, rows, st) : dg5_launch<64, DENSE_HALF>(p, rows, st);
+        case DENSE_ROPE:
+            if (wide) return dg5_launch<256, DENSE_ROPE>(p, rows, st);
+            return narrow ? dg5_launch<32, DENSE_ROPE>(p, rows, st) : dg5_launch<64, DENSE_ROPE>(p, rows, st);
         case DENSE_GATED: return wide ? dg5_launch<256, DENSE_GATED>(p, rows, st) : dg5_launch<64, DENSE_GATED>(p, rows, st);
         default: return wide ? dg5_launch<256, DENSE_QKV>(p, rows, st) : dg5_launch<64, DENSE_QKV>(p, rows, st);
     }
@@ -464,7 +513,7 @@ __global__ void __launch_bounds__(256) gate_f32_kernel(const float* __restrict__
 
 // gate_up: scratch of a gated product, float32 [rows][2 n]
 int launch_dense_gemm_f32(const DenseProduct& p, int rows, float* gate_up, cudaStream_t st) {
-    RB_REQUIRE(p.f32 && p.w && p.x && rows > 0 && p.epilogue != DENSE_QKV);
+    RB_REQUIRE(p.f32 && p.w && p.x && rows > 0 && p.epilogue != DENSE_QKV && p.epilogue != DENSE_ROPE);
     const bool gated = p.epilogue == DENSE_GATED;
     const int groups = p.groups ? p.groups : 1;
     RB_REQUIRE(gated ? (gate_up && p.a) : (p.epilogue == DENSE_HALF ? p.a != nullptr : p.y != nullptr));

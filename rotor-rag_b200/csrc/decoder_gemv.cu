@@ -373,7 +373,7 @@ static size_t dg_plan(const DenseProduct& p, int rows, int* grid, int* slots) {
 
 bool dense_gemv_supported(const DenseProduct& p, int rows) {
     int g, s;
-    if (p.groups > 65535 || p.epilogue == DENSE_QKV || (p.route && (p.route->top > EXPERT_TOP_MAX || p.route->top < 1))) return false;
+    if (p.groups > 65535 || p.epilogue == DENSE_QKV || p.epilogue == DENSE_ROPE || (p.route && (p.route->top > EXPERT_TOP_MAX || p.route->top < 1))) return false;
     return rows >= 1 && rows <= DENSE_FEW_ROWS && p.n > 0 && p.k > 0 && dg_plan(p, rows, &g, &s) <= DG_SMEM_MAX;
 }
 
