@@ -316,43 +316,45 @@ __device__ __forceinline__ float gate_act(int act, float z) { return act == ACT_
 __device__ __forceinline__ void route_row(const Routing& r, int row, int lane, int& sel, float& w) {
     const int experts = r.experts, top = r.top;
     auto logit = [&](int e) { return __ldcg(r.logits + (size_t)row * r.ld + e) + (r.bias ? __ldg(r.bias + e) : 0.f); };
-    float last = INFINITY, mine = -INFINITY, first = 0.f;
-    int last_i = -1;
     constexpr int KEPT = 4;  // logits per lane that stay in registers
     float kept[KEPT];
 #pragma unroll
     for (int j = 0; j < KEPT; ++j) kept[j] = lane + 32 * j < experts ? logit(lane + 32 * j) : -INFINITY;
+    // unsigned keys in the order of the values; what is not a number comes last
+    auto key_of = [](float v) {
+        const unsigned u = __float_as_uint(v);
+        return v != v ? 0u : (u & 0x80000000u ? ~u : u | 0x80000000u);
+    };
+    unsigned last = 0xffffffffu;
+    int last_i = -1;
+    float mine = -INFINITY, first = 0.f;
     sel = 0;
     for (int k = 0; k < top; ++k) {
-        float best = -INFINITY;
+        unsigned best = 0u;
         int best_i = 0x7fffffff;
-        auto offer = [&](int e, float v) {
-            if ((v < last || (v == last && e > last_i)) && (v > best || (v == best && e < best_i))) {
-                best = v;
+        float value = -INFINITY;
+        auto offer = [&](int e, float v) {  // (in order of e)
+            const unsigned q = key_of(v);
+            if ((q < last || (q == last && e > last_i)) && (best_i == 0x7fffffff || q > best)) {
+                best = q;
                 best_i = e;
+                value = v;
             }
         };
 #pragma unroll
         for (int j = 0; j < KEPT; ++j)
             if (lane + 32 * j < experts) offer(lane + 32 * j, kept[j]);
         for (int e = lane + 32 * KEPT; e < experts; e += 32) offer(e, logit(e));
-#pragma unroll
-        for (int o = 16; o > 0; o >>= 1) {
-            const float v = __shfl_xor_sync(0xffffffffu, best, o);
-            const int i = __shfl_xor_sync(0xffffffffu, best_i, o);
-            if (v > best || (v == best && i < best_i)) {
-                best = v;
-                best_i = i;
-            }
-        }
-        if (best_i >= experts) best_i = 0;  // (logits that are not numbers)
-        if (k == 0) first = best;
+        const unsigned top_key = __reduce_max_sync(0xffffffffu, best);
+        const int top_i = __reduce_min_sync(0xffffffffu, best == top_key ? best_i : 0x7fffffff);
+        const float top_v = __shfl_sync(0xffffffffu, value, top_i & 31);  // (expert e is lane e % 32's)
+        if (k == 0) first = top_v;
         if (lane == k) {
-            sel = best_i;
-            mine = best;
+            sel = min(top_i, experts - 1);
+            mine = top_v;
         }
-        last = best;
-        last_i = best_i;
+        last = top_key;
+        last_i = top_i;
     }
     const float e = lane < top ? expf(mine - first) : 0.f;
     w = e / warp_sum(e);
@@ -365,7 +367,8 @@ __device__ __forceinline__ void route_row(const Routing& r, int row, int lane, i
 template <int S>
 struct StreamGroup {
     float4 y, x[S ? S : 1];  // (a first stage keeps the embedding's columns in y)
-    // slot, slot_w: the row's part of slot_of and slot_w, wherever it lies
+    // slot, slot_w: the row's part of slot_of and slot_w, wherever it lies (SLOTS: there may be any)
+    template <bool SLOTS>
     __device__ __forceinline__ void load(const StreamStage& p, int row, int g, const int* slot, const float* slot_w) {
         if (p.ids) {
             long long id = p.ids[row];
@@ -381,11 +384,11 @@ struct StreamGroup {
             y.z += w * v.z;
             y.w += w * v.w;
         };
-        if (p.y2) add(__ldcg(reinterpret_cast<const float4*>(p.y2 + (size_t)row * p.ld) + g), 1.f);
-        if (p.slots && p.slots_f32) {
+        if (S <= 1 && p.y2) add(__ldcg(reinterpret_cast<const float4*>(p.y2 + (size_t)row * p.ld) + g), 1.f);
+        if (SLOTS && p.slots && p.slots_f32) {
             for (int k = 0; k < p.top; ++k)
                 add(__ldcg(reinterpret_cast<const float4*>(static_cast<const float*>(p.slots) + (size_t)slot[k] * p.ld) + g), slot_w[k]);
-        } else if (p.slots) {
+        } else if (SLOTS && p.slots) {
             constexpr int U = 4;  // slots requested together
             for (int k0 = 0; k0 < p.top; k0 += U) {
                 uint2 v[U];

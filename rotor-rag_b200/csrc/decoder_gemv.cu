@@ -8,8 +8,8 @@
 // one 128-bit weight load per lane; loads run a batch ahead of the arithmetic, and the first batches
 // are requested before the programmatic-launch wait.
 //
-// Variants (MODE): products of two normed rows of one stage (the second a small one: a router), one product
-// per group (grid.y: heads), and a token's experts -- the gated product of each (token, choice) with the
+// Variants (MODE): products of two normed rows of one stage (the second a small one: a router), of float32 rows
+// normed on the way, one product per group (grid.y: heads), and a token's experts -- the gated product of each (token, choice) with the
 // expert's weights (grid.y; every CTA makes the choice itself from the router's outputs), and the weighted
 // sum of their down products as one product whose K runs over the choices.
 #include "decoder.cuh"
@@ -27,7 +27,7 @@ struct DenseGemvArgs {
     Routing route;
     int has_stage, rows, slots, max_rows;
 };
-enum { GV_PLAIN = 0, GV_DUAL = 1, GV_GROUPS = 2, GV_EXPERT_UP = 3, GV_EXPERT_DOWN = 4 };
+enum { GV_PLAIN = 0, GV_DUAL = 1, GV_GROUPS = 2, GV_EXPERT_UP = 3, GV_EXPERT_DOWN = 4, GV_NORMED = 5 };
 
 // Column i (a multiple of 4) of a staged row: the two halves of a lane's eight columns sit 128 floats
 // apart, which makes both 128-bit reads of a unit free of bank conflicts.
@@ -146,14 +146,14 @@ __global__ void __launch_bounds__(DG_THREADS, R <= 2 ? 2 : 1) dense_gemv_kernel(
                 StreamGroup<S> sg[SG];
 #pragma unroll
                 for (int i = 0; i < SG; ++i)
-                    if (g0 + i * DG_THREADS < n4) sg[i].load(s, r, g0 + i * DG_THREADS, s.slot_of + (size_t)r * s.top, s.slot_w + (size_t)r * s.top);
+                    if (g0 + i * DG_THREADS < n4) sg[i].template load<false>(s, r, g0 + i * DG_THREADS, nullptr, nullptr);
 #pragma unroll
                 for (int i = 0; i < SG; ++i) {
                     const int g = g0 + i * DG_THREADS;
                     float4 u = make_float4(0.f, 0.f, 0.f, 0.f);
                     if (g < n4) {
                         u = sg[i].finish(s, coef, r, g, g % gridDim.x == blockIdx.x);
-                        ss += s.norm_b ? u.x + u.y + u.z + u.w : u.x * u.x + u.y * u.y + u.z * u.z + u.w * u.w;
+                        ss += S == 1 && s.norm_b ? u.x + u.y + u.z + u.w : u.x * u.x + u.y * u.y + u.z * u.z + u.w * u.w;
                     }
                     if (g < (kx >> 2)) {
                         *reinterpret_cast<float4*>(xs + r * kx + dg_slot(g << 2)) = u;
@@ -163,7 +163,7 @@ __global__ void __launch_bounds__(DG_THREADS, R <= 2 ? 2 : 1) dense_gemv_kernel(
             }
             ss = block_sum_alt(ss, red, k);
             float mean = 0.f;
-            if (s.norm_b) {
+            if (S == 1 && s.norm_b) {
                 mean = ss / (float)s.n;
                 ss = 0.f;
                 for (int g = threadIdx.x; g < n4; g += DG_THREADS)
@@ -174,7 +174,7 @@ __global__ void __launch_bounds__(DG_THREADS, R <= 2 ? 2 : 1) dense_gemv_kernel(
             auto scale = [&](int g, const float4 w) {  // own groups
                 float4* q = reinterpret_cast<float4*>(xs + r * kx + dg_slot(g << 2));
                 const float4 u = *q;
-                float4 v = norm_group(u, mean, inv, w, s.norm_b, g);
+                float4 v = norm_group(u, mean, inv, w, S == 1 ? s.norm_b : nullptr, g);
                 if (!p.f32) v = make_float4(round_bf16(v.x), round_bf16(v.y), round_bf16(v.z), round_bf16(v.w));
                 *q = v;
                 if constexpr (MODE == GV_DUAL) {
@@ -196,54 +196,71 @@ __global__ void __launch_bounds__(DG_THREADS, R <= 2 ? 2 : 1) dense_gemv_kernel(
                 scale(g, __ldg(reinterpret_cast<const float4*>(s.norm) + g));
         }
     } else {
-        constexpr int XG = 4;
-        const bool wide = p.f32 || p.x_raw;  // float32 rows
-        int k = 0;
-        for (int q = 0; q < R * segs; ++q) {
-            size_t at = (size_t)q * p.ldx;  // (one row: its choices)
-            if constexpr (MODE == GV_GROUPS) at += (size_t)y * p.gx_col;
-            if constexpr (MODE == GV_EXPERT_UP) at = (size_t)(y / a.route.top) * p.ldx;
-            if constexpr (MODE == GV_EXPERT_DOWN) at += (size_t)y * a.route.top * p.ldx;
-            const float gain = MODE == GV_EXPERT_DOWN ? s_weight[q] : 1.f;
-            float ss = 0.f;
-            for (int g0 = threadIdx.x; g0 < (kx >> 2); g0 += XG * DG_THREADS) {
+        constexpr int XG = 4;  // column groups per thread requested together
+        constexpr bool RAW = MODE == GV_GROUPS || MODE == GV_NORMED;
+        const bool wide = p.f32 || (RAW && p.x_raw);  // float32 rows
+        const int n4 = kx >> 2;
+        // first element of staged row q (of x's rows; of a token's choices)
+        auto row_of = [&](int q) {
+            if constexpr (MODE == GV_GROUPS) return (size_t)q * p.ldx + (size_t)y * p.gx_col;
+            if constexpr (MODE == GV_EXPERT_UP) return (size_t)(y / a.route.top) * p.ldx;
+            if constexpr (MODE == GV_EXPERT_DOWN) return ((size_t)y * a.route.top + q) * p.ldx;
+            return (size_t)q * p.ldx;
+        };
+        auto request = [&](int q, int g) {
+            if ((g << 2) >= p.k) return make_float4(0.f, 0.f, 0.f, 0.f);
+            if (wide) return __ldcg(reinterpret_cast<const float4*>(static_cast<const float*>(p.x) + row_of(q)) + g);
+            return bf16x4_to_float4(__ldcg(reinterpret_cast<const uint2*>(static_cast<const __nv_bfloat16*>(p.x) + row_of(q)) + g));
+        };
+        auto put = [&](int q, int g, float4 v) {
+            const int c = g << 2;
+            if (c + 1 >= p.k) v.y = 0.f;  // (pad columns of the row may hold another product's values)
+            if (c + 2 >= p.k) v.z = 0.f;
+            if (c + 3 >= p.k) v.w = 0.f;
+            if constexpr (MODE == GV_EXPERT_DOWN) {
+                const float gain = s_weight[q];
+                v = make_float4(v.x * gain, v.y * gain, v.z * gain, v.w * gain);
+            }
+            if (MODE == GV_GROUPS && p.x_raw && !p.f32) v = make_float4(round_bf16(v.x), round_bf16(v.y), round_bf16(v.z), round_bf16(v.w));
+            *reinterpret_cast<float4*>(xs + q * kx + dg_slot(c)) = v;
+        };
+        if constexpr (MODE == GV_EXPERT_DOWN) {  // short rows: requests run on from one to the next
+            for (int i0 = threadIdx.x; i0 < segs * n4; i0 += XG * DG_THREADS) {
                 float4 f[XG];
 #pragma unroll
-                for (int i = 0; i < XG; ++i) {
-                    const int g = g0 + i * DG_THREADS;
-                    f[i] = make_float4(0.f, 0.f, 0.f, 0.f);
-                    if ((g << 2) >= p.k) continue;
-                    if (wide)
-                        f[i] = __ldcg(reinterpret_cast<const float4*>(static_cast<const float*>(p.x) + at) + g);
-                    else
-                        f[i] = bf16x4_to_float4(__ldcg(reinterpret_cast<const uint2*>(static_cast<const __nv_bfloat16*>(p.x) + at) + g));
-                }
+                for (int i = 0; i < XG; ++i)
+                    if (i0 + i * DG_THREADS < segs * n4) f[i] = request((i0 + i * DG_THREADS) / n4, (i0 + i * DG_THREADS) % n4);
 #pragma unroll
-                for (int i = 0; i < XG; ++i) {
-                    const int c = (g0 + i * DG_THREADS) << 2;
-                    if (c >= kx) continue;
-                    if (c + 1 >= p.k) f[i].y = 0.f;  // (pad columns of the row may hold another product's values)
-                    if (c + 2 >= p.k) f[i].z = 0.f;
-                    if (c + 3 >= p.k) f[i].w = 0.f;
-                    if constexpr (MODE == GV_EXPERT_DOWN) f[i] = make_float4(f[i].x * gain, f[i].y * gain, f[i].z * gain, f[i].w * gain);
-                    if (p.x_raw) {
-                        if (p.x_norm)
-                            ss += f[i].x * f[i].x + f[i].y * f[i].y + f[i].z * f[i].z + f[i].w * f[i].w;
-                        else if (!p.f32)
-                            f[i] = make_float4(round_bf16(f[i].x), round_bf16(f[i].y), round_bf16(f[i].z), round_bf16(f[i].w));
-                    }
-                    *reinterpret_cast<float4*>(xs + q * kx + dg_slot(c)) = f[i];
-                }
+                for (int i = 0; i < XG; ++i)
+                    if (i0 + i * DG_THREADS < segs * n4) put((i0 + i * DG_THREADS) / n4, (i0 + i * DG_THREADS) % n4, f[i]);
             }
-            if (!p.x_norm) continue;
-            ss = block_sum_alt(ss, red, k);
-            const float inv = 1.0f / sqrtf(ss / (float)p.k + p.x_eps);
-            for (int g = threadIdx.x; g < (kx >> 2); g += DG_THREADS) {  // own groups
-                if ((g << 2) >= p.k) continue;
-                float4* v = reinterpret_cast<float4*>(xs + q * kx + dg_slot(g << 2));
-                float4 u = norm_group(*v, 0.f, inv, p.x_norm, nullptr, g);
-                if (!p.f32) u = make_float4(round_bf16(u.x), round_bf16(u.y), round_bf16(u.z), round_bf16(u.w));
-                *v = u;
+        } else {
+            for (int r = 0; r < R; ++r)
+                for (int g0 = threadIdx.x; g0 < n4; g0 += XG * DG_THREADS) {
+                    float4 f[XG];
+#pragma unroll
+                    for (int i = 0; i < XG; ++i) f[i] = request(r, g0 + i * DG_THREADS);
+#pragma unroll
+                    for (int i = 0; i < XG; ++i)
+                        if (g0 + i * DG_THREADS < n4) put(r, g0 + i * DG_THREADS, f[i]);
+                }
+        }
+        if constexpr (MODE == GV_NORMED) {
+            int k = 0;
+            for (int r = 0; r < R; ++r) {
+                float ss = 0.f;
+                for (int g = threadIdx.x; g < n4; g += DG_THREADS) {  // own groups
+                    const float4 u = *reinterpret_cast<const float4*>(xs + r * kx + dg_slot(g << 2));
+                    ss += u.x * u.x + u.y * u.y + u.z * u.z + u.w * u.w;
+                }
+                ss = block_sum_alt(ss, red, k);
+                const float inv = 1.0f / sqrtf(ss / (float)p.k + p.x_eps);
+                for (int g = threadIdx.x; (g << 2) < p.k; g += DG_THREADS) {
+                    float4* v = reinterpret_cast<float4*>(xs + r * kx + dg_slot(g << 2));
+                    float4 u = norm_group(*v, 0.f, inv, p.x_norm, nullptr, g);
+                    if (!p.f32) u = make_float4(round_bf16(u.x), round_bf16(u.y), round_bf16(u.z), round_bf16(u.w));
+                    *v = u;
+                }
             }
         }
     }
@@ -355,6 +372,7 @@ __global__ void __launch_bounds__(DG_THREADS, R <= 2 ? 2 : 1) dense_gemv_kernel(
 static int dg_mode(const DenseProduct& p) {
     if (p.route) return p.epilogue == DENSE_GATED ? GV_EXPERT_UP : GV_EXPERT_DOWN;
     if (p.groups) return GV_GROUPS;
+    if (p.x_norm) return GV_NORMED;
     return p.stage && p.stage->norm2 ? GV_DUAL : GV_PLAIN;
 }
 
@@ -374,6 +392,8 @@ static size_t dg_plan(const DenseProduct& p, int rows, int* grid, int* slots) {
 bool dense_gemv_supported(const DenseProduct& p, int rows) {
     int g, s;
     if (p.groups > 65535 || p.epilogue == DENSE_QKV || p.epilogue == DENSE_ROPE || (p.route && (p.route->top > EXPERT_TOP_MAX || p.route->top < 1))) return false;
+    // (what a stage adds up and norms beyond one stream's share is the stage kernel's)
+    if (p.stage && (p.stage->slots || (p.stage->streams != 1 && (p.stage->norm_b || p.stage->y2)))) return false;
     return rows >= 1 && rows <= DENSE_FEW_ROWS && p.n > 0 && p.k > 0 && dg_plan(p, rows, &g, &s) <= DG_SMEM_MAX;
 }
 
@@ -387,7 +407,7 @@ static int dg_configure_all() {
     int rc;
     if ((rc = dg_configure<R, 0, GV_PLAIN>()) || (rc = dg_configure<R, 1, GV_PLAIN>()) || (rc = dg_configure<R, 2, GV_PLAIN>()) ||
         (rc = dg_configure<R, 3, GV_PLAIN>()) || (rc = dg_configure<R, 4, GV_PLAIN>()) || (rc = dg_configure<R, 1, GV_DUAL>()) ||
-        (rc = dg_configure<R, 1, GV_GROUPS>()))
+        (rc = dg_configure<R, 1, GV_GROUPS>()) || (rc = dg_configure<R, 1, GV_NORMED>()))
         return rc;
     return ROTOR_B200_OK;
 }
@@ -403,6 +423,7 @@ template <int R>
 static int dg_launch(const DenseGemvArgs& a, int mode, int grid, size_t smem, cudaStream_t st) {
     const dim3 g(grid, mode == GV_GROUPS ? a.p.groups : 1), b(DG_THREADS);
     if (mode == GV_GROUPS) return launch_chained(dense_gemv_kernel<R, 1, GV_GROUPS>, g, b, smem, st, 1, a);
+    if (mode == GV_NORMED) return launch_chained(dense_gemv_kernel<R, 1, GV_NORMED>, g, b, smem, st, 1, a);
     if (mode == GV_DUAL) return launch_chained(dense_gemv_kernel<R, 1, GV_DUAL>, g, b, smem, st, 1, a);
     switch (a.has_stage ? a.st.streams : 1) {
         case 1: return launch_chained(dense_gemv_kernel<R, 1, GV_PLAIN>, g, b, smem, st, 1, a);
@@ -420,7 +441,8 @@ int launch_dense_gemv(const DenseProduct& p, int rows, cudaStream_t st) {
     RB_REQUIRE(p.epilogue == DENSE_GATED || mode == GV_GROUPS ? p.a != nullptr : p.y != nullptr);
     RB_REQUIRE(mode != GV_GROUPS || (p.epilogue == DENSE_HALF && p.gx_col % 4 == 0 && !p.stage));
     RB_REQUIRE(!p.route || (p.route->logits && p.route->top <= p.route->experts && !p.stage && !p.x_norm));
-    RB_REQUIRE(!p.x_norm || p.x_raw);
+    RB_REQUIRE(!p.x_norm || (p.x_raw && !p.stage && mode == GV_NORMED));
+    RB_REQUIRE(!p.x_raw || mode == GV_NORMED || mode == GV_GROUPS);
     DenseGemvArgs a = {};
     a.p = p;
     if (p.route) a.route = *p.route;

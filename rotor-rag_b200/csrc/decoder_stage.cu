@@ -33,7 +33,7 @@ __global__ void __launch_bounds__(256) stream_stage_kernel(const __grid_constant
             StreamGroup<S> sg[U];
 #pragma unroll
             for (int i = 0; i < U; ++i)
-                if (g0 + i * (int)blockDim.x < n4) sg[i].load(p, src, g0 + i * blockDim.x, slot, slot_w);
+                if (g0 + i * (int)blockDim.x < n4) sg[i].template load<true>(p, src, g0 + i * blockDim.x, slot, slot_w);
 #pragma unroll
             for (int i = 0; i < U; ++i) {
                 const int g = g0 + i * blockDim.x;

@@ -12,8 +12,6 @@
 //   bf16:    16 heads a tile are the M of mma.m16n8k16: warps split the positions and halves of a row for the
 //            scores and the latent columns for the sums
 //   float32: the FP32 pipe, eight heads a tile
-#include <type_traits>
-
 #include "decoder.cuh"
 
 namespace rb {
@@ -38,16 +36,28 @@ __device__ __forceinline__ void la_store2(float* p, const float2 v) { *reinterpr
 // One warp makes a cache row from its raw projection: put(column, value pair) for all kp + rp columns.
 template <typename F>
 __device__ __forceinline__ void latent_cache_row(const LatentShape& s, const float* raw, const float* norm, const float2* rope, int lane, F put) {
+    constexpr int U = 8;  // column pairs per lane that stay in registers
+    float2 keep[U];
     float ss = 0.f;
-    for (int c = lane; c < s.rank; c += 32) {
-        const float v = __ldcg(raw + c);
-        ss += v * v;
+    auto pair = [&](int c) {  // (the columns between rank and kp are zeros)
+        return 2 * c < s.kp ? __ldcg(reinterpret_cast<const float2*>(raw) + c) : make_float2(0.f, 0.f);
+    };
+#pragma unroll
+    for (int u = 0; u < U; ++u) keep[u] = pair(lane + 32 * u);
+#pragma unroll
+    for (int u = 0; u < U; ++u) ss += keep[u].x * keep[u].x + keep[u].y * keep[u].y;
+    for (int c = lane + 32 * U; 2 * c < s.kp; c += 32) {
+        const float2 v = pair(c);
+        ss += v.x * v.x + v.y * v.y;
     }
     const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)s.rank + s.eps);
-    for (int c = 2 * lane; c < s.kp; c += 64) {
-        const float2 v = __ldcg(reinterpret_cast<const float2*>(raw + c));
-        put(c, make_float2(c < s.rank ? v.x * inv * __ldg(norm + c) : 0.f, c + 1 < s.rank ? v.y * inv * __ldg(norm + c + 1) : 0.f));
-    }
+    auto scaled = [&](int c, const float2 v) {
+        if (2 * c < s.kp)
+            put(2 * c, make_float2(2 * c < s.rank ? v.x * inv * __ldg(norm + 2 * c) : 0.f, 2 * c + 1 < s.rank ? v.y * inv * __ldg(norm + 2 * c + 1) : 0.f));
+    };
+#pragma unroll
+    for (int u = 0; u < U; ++u) scaled(lane + 32 * u, keep[u]);
+    for (int c = lane + 32 * U; 2 * c < s.kp; c += 32) scaled(c, pair(c));
     for (int i = lane; i < (s.rp >> 1); i += 32) {
         const float2 v = __ldcg(reinterpret_cast<const float2*>(raw + s.kp) + i);
         put(s.kp + 2 * i, 2 * i < s.rot ? rot_pair(v, __ldg(rope + i)) : make_float2(0.f, 0.f));
@@ -238,22 +248,39 @@ __device__ __forceinline__ void la_merge(const LatentAttn& p, const float* po, i
 template <typename T>
 __device__ __forceinline__ void la_queries(const LatentAttn& p, T* qs, int stride, int h0, int nh, int tile_heads, int row, const float2* rope) {
     const LatentShape& s = p.s;
-    const int W = s.kp + s.rp, half = W >> 1;
-    const T* q = static_cast<const T*>(p.q_abs) + (size_t)row * s.heads * W;
-    typedef typename std::conditional<sizeof(T) == 2, uint32_t, uint2>::type Pair;
-    for (int i = threadIdx.x; i < tile_heads * half; i += LA_THREADS) {
-        const int h = i / half, c = (i - h * half) * 2;
-        Pair v = {};
-        if (h < nh && (c < s.kp || !p.q_raw))
-            v = __ldcg(reinterpret_cast<const Pair*>(q + (size_t)(h0 + h) * W + c));
-        *reinterpret_cast<Pair*>(qs + h * stride + c) = v;
-        if (h < nh && c >= s.kp && p.q_raw) {
-            const int r = (c - s.kp) >> 1;
-            if (2 * r < s.rot) {
-                const float2 x = __ldcg(reinterpret_cast<const float2*>(p.q_raw + (size_t)row * p.ldq + (size_t)(h0 + h) * (s.dp + s.rp) + s.dp) + r);
-                la_store2(qs + h * stride + c, rot_pair(x, __ldg(rope + r)));
-            }
+    constexpr int PIECE = 16 / (int)sizeof(T), U = 3;  // pieces per thread requested together
+    const int W = s.kp + s.rp, from = p.q_raw ? s.kp : W, pieces = from / PIECE, total = tile_heads * pieces;
+    const T* q = static_cast<const T*>(p.q_abs) + ((size_t)row * s.heads + h0) * W;
+    // the rotated part from the raw projections: requested first, turned last
+    const int pairs = p.q_raw ? s.rp >> 1 : 0, rots = tile_heads * pairs;
+    float2 raw = make_float2(0.f, 0.f), cs = raw;
+    auto rot_of = [&](int i, float2& x, float2& t) {
+        const int h = i / pairs, r = i - h * pairs;
+        x = t = make_float2(0.f, 0.f);
+        if (h < nh && 2 * r < s.rot) {
+            x = __ldcg(reinterpret_cast<const float2*>(p.q_raw + (size_t)row * p.ldq + (size_t)(h0 + h) * (s.dp + s.rp) + s.dp) + r);
+            t = __ldg(rope + r);
         }
+    };
+    if ((int)threadIdx.x < rots) rot_of(threadIdx.x, raw, cs);
+    for (int i0 = threadIdx.x; i0 < total; i0 += U * LA_THREADS) {
+        uint4 v[U];
+#pragma unroll
+        for (int u = 0; u < U; ++u) {
+            const int i = i0 + u * LA_THREADS, h = i / pieces, c = i - h * pieces;
+            v[u] = make_uint4(0u, 0u, 0u, 0u);
+            if (i < total && h < nh) v[u] = __ldcg(reinterpret_cast<const uint4*>(q + (size_t)h * W) + c);
+        }
+#pragma unroll
+        for (int u = 0; u < U; ++u) {
+            const int i = i0 + u * LA_THREADS, h = i / pieces, c = i - h * pieces;
+            if (i < total) *reinterpret_cast<uint4*>(qs + h * stride + c * PIECE) = v[u];
+        }
+    }
+    for (int i = threadIdx.x; i < rots; i += LA_THREADS) {
+        if (i != (int)threadIdx.x) rot_of(i, raw, cs);
+        const int h = i / pairs, r = i - h * pairs;
+        la_store2(qs + h * stride + s.kp + 2 * r, rot_pair(raw, cs));
     }
 }
 
