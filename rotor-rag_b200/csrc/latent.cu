@@ -316,10 +316,13 @@ __global__ void __launch_bounds__(LA_THREADS) latent_attn_mma_kernel(const __gri
     const int skip = p.dkv ? run.pos : -1;
 
     if (p.early && run.t0 < run.t1) run.load(kv, run.t0, TK, skip);
+    if (p.dkv && warp == 0) {  // constants the new row needs
+        for (int c = lane * 32; c < s.rank; c += 32 * 32) prefetch_l2(p.dkv_norm + c);
+        if (lane * 16 < (s.rot >> 1)) prefetch_l2(rope + lane * 16);
+    }
     pdl_wait();
     pdl_trigger();
     if (!p.early && run.t0 < run.t1) run.load(kv, run.t0, TK, skip);
-    la_queries(p, qs, ws, h0, nh, LA_HEADS, run.row, rope);
     const bool owner = p.dkv && run.t0 <= run.pos && run.pos < run.t1;  // (the last position of the run)
     if (owner && warp == 0) {
         const int k0 = (run.pos - run.t0) / TK * TK + run.t0;
@@ -330,8 +333,9 @@ __global__ void __launch_bounds__(LA_THREADS) latent_attn_mma_kernel(const __gri
             if (k0 == run.t0) la_store2(stage + c, x);
             if (blockIdx.y == 0 || k0 != run.t0) la_store2(dst + c, x);
         });
-        __threadfence();
+        if (k0 != run.t0) __threadfence();
     }
+    la_queries(p, qs, ws, h0, nh, LA_HEADS, run.row, rope);
     if (tid < LA_HEADS) {
         ml[tid] = -INFINITY;
         ml[LA_HEADS + tid] = 0.f;
